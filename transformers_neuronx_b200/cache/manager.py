@@ -41,16 +41,20 @@ def _element_size(dtype) -> int:
 class PagedKVNeed:
     """Keys and values of every position (window None) or of the last `window` positions, in the
     engine's activation type: one tensor [pages, 2 (key, value), n_kv_heads, page_size, head_dim].
+    `keep_first`: with a window, the first positions stay readable for good, and their pages with them.
     `chunk`: queries read the keys of their own block of `chunk` positions only, so the pages of the blocks
     before the running one are given back."""
     n_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     chunk: Optional[int] = None
+    keep_first: int = 0
     clear_on_admission = False
 
     @property
     def group_key(self):
+        if self.keep_first:
+            return ("paged", self.window, self.chunk, self.keep_first)
         return ("paged", self.window) if self.chunk is None else ("paged", self.window, self.chunk)
 
     def make_storage(self, page_size, num_pages, max_slots, act_dtype, device):
@@ -87,6 +91,7 @@ class GroupInfo:
     cache_ids: List[int]
     window: Optional[int] = None
     chunk: Optional[int] = None
+    keep_first: int = 0
 
     @property
     def releases(self) -> bool:
@@ -109,7 +114,7 @@ def group_needs(needs: Dict[int, object]) -> List[GroupInfo]:
         k = need.group_key
         if k not in groups:
             groups[k] = GroupInfo(key=k, cache_ids=[], window=getattr(need, "window", None),
-                                  chunk=getattr(need, "chunk", None))
+                                  chunk=getattr(need, "chunk", None), keep_first=getattr(need, "keep_first", 0))
         groups[k].cache_ids.append(cid)
     return list(groups.values())
 
@@ -203,11 +208,12 @@ class CacheManager:
         n = 0
         for g, pool, table in zip(self.paged_groups, self.pools, r.tables):
             first = min(self._first_needed_block(g, r.length), len(table))
-            gone = [p for p in table[:first] if p >= 0]
+            kept = min(-(-g.keep_first // self.page_size), first)     # the blocks of the first tokens stay
+            gone = [p for p in table[kept:first] if p >= 0]
             if gone:
                 pool.free(gone, rid)
                 n += len(gone)
-                for b in range(first):
+                for b in range(kept, first):
                     table[b] = -1
         return n
 

@@ -2,9 +2,10 @@
 // of its request streamed from the pages named by its block table.  Memory-bound: every key and
 // value of the live requests is read once per layer and step.
 //
-//   s_j = scale * <q, k_j>  (32-bit),  out = sum_j exp(s_j - max) v_j / sum_j exp(s_j - max)
+//   s_j = scale * <q, k_j>  (32-bit; less a distance bias where one is given),  out = sum_j exp(s_j - max) v_j / sum_j exp(s_j - max)
 //
-// Grid (heads, rows, splits): a CTA takes one (row, head) and one contiguous range of pages; its
+// Grid (heads, rows, splits): a CTA takes one (row, head) and one contiguous range of the pages that hold visible keys
+// (behind a window the pages before it are not counted; those of the first keys that are kept come first); its
 // four, eight or sixteen warps take pages of the range in turn and keep an online softmax each (half a page at a
 // time, the next half's loads in flight meanwhile).  A lane owns eight
 // consecutive dims of the head (one 16-byte load per key) of some of the keys of a page, so a page
@@ -34,6 +35,8 @@ struct DecodeParams {
     int n_heads, n_kv_heads, head_dim;
     int window;                      // the mask rule of common.cuh: first_visible_key
     float scale;
+    int keep_first;                  // with a window: the first positions that stay visible
+    DistanceBias bias;
     int n_splits, pages_per_split;
     float* scratch;                  // [rows][heads][splits][head_dim + 2]
     int* counters;                   // [rows][heads], zero between calls
@@ -53,7 +56,8 @@ struct DecodeParams {
 // value loaded feeds REP dot products and accumulators; with one block per query head the heads of a group each
 // stream the group's pages (measured at batch 64 with 4 query heads a key/value head: 308 us a layer where the pages'
 // own streaming takes 81).
-template <int LPK, int E, int WARPS, int REP>
+// BIAS: the scores lose a distance bias (per head; a logarithm a key).
+template <int LPK, int E, int WARPS, int REP, bool BIAS>
 __global__ void __launch_bounds__(WARPS * 32)
 attention_decode_kernel(const DecodeParams p) {
     constexpr int KPL = 32 / LPK;
@@ -111,14 +115,25 @@ attention_decode_kernel(const DecodeParams p) {
             for (int i = 0; i < 8; ++i) acc[x][e][i] = 0.f;
     }
 
+    float bias_mul[REP], bias_rate[REP];                         // of a logarithm to base 2
+    if constexpr (BIAS) {
+#pragma unroll
+        for (int x = 0; x < REP; ++x) {
+            bias_mul[x] = p.bias.mul[h0 + x] * 0.6931471805599453f;
+            bias_rate[x] = p.bias.rate[h0 + x];
+        }
+    }
+
     const int n_pages = (kv_len + PAGE - 1) / PAGE;
-    const int page_lo = max(split * p.pages_per_split, first_key / PAGE);
-    const int page_hi = min(n_pages, (split + 1) * p.pages_per_split);
+    // pages are numbered along the walk over the visible ones
+    const BlockWalk walk = walk_blocks(first_key, p.keep_first, PAGE);
+    const int page_lo = split * p.pages_per_split;
+    const int page_hi = min(walk.count(n_pages - 1), (split + 1) * p.pages_per_split);
     const size_t head_block = (size_t)PAGE * d;
 
     // With the append fused in, the cache holds the keys before this token's own; its own key and
     // value come from k_new / v_new.
-    const bool own_here = p.k_new != nullptr && (pos / PAGE) / p.pages_per_split == split;    // one answer for the CTA
+    const bool own_here = p.k_new != nullptr && walk.place(pos / PAGE) / p.pages_per_split == split;    // one answer for the CTA
     const int cached_len = p.k_new != nullptr ? pos : kv_len;
     // The warp's pages (page_lo + warp, + WARPS, ...) are taken in chunks of CG key groups, i.e. CH = CG * E
     // warp-wide loads of keys and as many of values: half a page of the widest heads, a whole page
@@ -131,8 +146,7 @@ attention_decode_kernel(const DecodeParams p) {
     const int my_pages = page_hi > page_lo + warp ? (page_hi - page_lo - warp + WARPS - 1) / WARPS : 0;
     const int n_chunks = my_pages * CPP;
     auto issue = [&](int t, uint4 (&kb)[CH], uint4 (&vb)[CH]) {
-        const int pg = page_lo + warp + (t / CPP) * WARPS;
-        const int page = bt[pg];
+        const int page = bt[walk.at(page_lo + warp + (t / CPP) * WARPS)];
         const h16* kbase = p.cache + (((size_t)page * 2 + 0) * p.n_kv_heads + kvh) * head_block;
         const h16* vbase = p.cache + (((size_t)page * 2 + 1) * p.n_kv_heads + kvh) * head_block;
         const int g0 = (t % CPP) * CG;
@@ -152,7 +166,7 @@ attention_decode_kernel(const DecodeParams p) {
             }
     };
     auto consume = [&](int t, uint4 (&kb)[CH], uint4 (&vb)[CH]) {
-        const int pg = page_lo + warp + (t / CPP) * WARPS;
+        const int pg = walk.at(page_lo + warp + (t / CPP) * WARPS);
         const int g0 = (t % CPP) * CG;
         float s[REP][CG];
         float chunk_max[REP];
@@ -161,7 +175,8 @@ attention_decode_kernel(const DecodeParams p) {
 #pragma unroll
         for (int g = 0; g < CG; ++g) {
             const int j = pg * PAGE + (g0 + g) * KPL + kgrp;
-            const bool seen = j >= first_key && j < cached_len;          // the same for every head
+            const bool seen = (j >= first_key || j < p.keep_first) && j < cached_len;    // the same for every head
+            const float dist = (float)(pos - j);
 #pragma unroll
             for (int x = 0; x < REP; ++x) {
                 float dot = 0.f;
@@ -179,6 +194,7 @@ attention_decode_kernel(const DecodeParams p) {
                 }
 #pragma unroll
                 for (int o = LPK / 2; o > 0; o >>= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
+                if constexpr (BIAS) dot -= bias_mul[x] * log2_approx(fmaf(bias_rate[x], dist, 1.f));
                 s[x][g] = seen ? dot : -INFINITY;
                 chunk_max[x] = fmaxf(chunk_max[x], s[x][g]);
             }
@@ -405,24 +421,30 @@ attention_decode_kernel(const DecodeParams p) {
 // E = 1 and at most 16 lanes a key, where the registers allow it; 8 otherwise).
 // rep > 1 (2 or 4, only where gqa_rep() below says so): a block takes the rep query heads of a key/value head, with
 // 4 or 8 warps (their accumulators leave no registers for 16).
-template <int LPK, int E>
-int launch_decode(int warps, int rep, dim3 grid, cudaStream_t stream, const DecodeParams& p) {
+template <int LPK, int E, bool BIAS>
+int launch_decode_as(int warps, int rep, dim3 grid, cudaStream_t stream, const DecodeParams& p) {
     if constexpr (E == 1 && (LPK == 8 || LPK == 16)) {
         if (rep == 4) {
-            if (warps >= 8) return tnx_launch_in_order(attention_decode_kernel<LPK, E, 8, 4>, grid, dim3(8 * 32), 0, stream, p);
-            return tnx_launch_in_order(attention_decode_kernel<LPK, E, 4, 4>, grid, dim3(4 * 32), 0, stream, p);
+            if (warps >= 8) return tnx_launch_in_order(attention_decode_kernel<LPK, E, 8, 4, BIAS>, grid, dim3(8 * 32), 0, stream, p);
+            return tnx_launch_in_order(attention_decode_kernel<LPK, E, 4, 4, BIAS>, grid, dim3(4 * 32), 0, stream, p);
         }
         if (rep == 2) {
-            if (warps >= 8) return tnx_launch_in_order(attention_decode_kernel<LPK, E, 8, 2>, grid, dim3(8 * 32), 0, stream, p);
-            return tnx_launch_in_order(attention_decode_kernel<LPK, E, 4, 2>, grid, dim3(4 * 32), 0, stream, p);
+            if (warps >= 8) return tnx_launch_in_order(attention_decode_kernel<LPK, E, 8, 2, BIAS>, grid, dim3(8 * 32), 0, stream, p);
+            return tnx_launch_in_order(attention_decode_kernel<LPK, E, 4, 2, BIAS>, grid, dim3(4 * 32), 0, stream, p);
         }
     }
     if (rep != 1) return TNX_ERR_UNSUPPORTED;
     if constexpr (E == 1 && LPK <= 16) {
-        if (warps == 16) return tnx_launch_in_order(attention_decode_kernel<LPK, E, 16, 1>, grid, dim3(16 * 32), 0, stream, p);
+        if (warps == 16) return tnx_launch_in_order(attention_decode_kernel<LPK, E, 16, 1, BIAS>, grid, dim3(16 * 32), 0, stream, p);
     }
-    if (warps >= 8) return tnx_launch_in_order(attention_decode_kernel<LPK, E, 8, 1>, grid, dim3(8 * 32), 0, stream, p);
-    return tnx_launch_in_order(attention_decode_kernel<LPK, E, 4, 1>, grid, dim3(4 * 32), 0, stream, p);
+    if (warps >= 8) return tnx_launch_in_order(attention_decode_kernel<LPK, E, 8, 1, BIAS>, grid, dim3(8 * 32), 0, stream, p);
+    return tnx_launch_in_order(attention_decode_kernel<LPK, E, 4, 1, BIAS>, grid, dim3(4 * 32), 0, stream, p);
+}
+
+template <int LPK, int E>
+int launch_decode(int warps, int rep, dim3 grid, cudaStream_t stream, const DecodeParams& p) {
+    return p.bias.mul ? launch_decode_as<LPK, E, true>(warps, rep, grid, stream, p)
+                      : launch_decode_as<LPK, E, false>(warps, rep, grid, stream, p);
 }
 
 // How many query heads a block takes for these sizes: 4 where the query heads per key/value head are a multiple of 4
@@ -456,7 +478,8 @@ TNX_EXPORT int tnx_attention_decode_append(const void* q, int q_stride, void* ca
                                            void* out, int out_stride, int n_rows, int n_heads, int n_kv_heads, int head_dim,
                                            int page_size, int window, float scale, int n_splits, int pages_per_split,
                                            float* scratch, int* counters, const void* k_new, const void* v_new,
-                                           int kv_stride, int warps, int heads_per_block, cudaStream_t stream) {
+                                           int kv_stride, int warps, int heads_per_block, int keep_first,
+                                           const float* bias_mul, const float* bias_rate, cudaStream_t stream) {
     // heads_per_block: 1, or what tnx_attention_decode_heads_per_block answers for these sizes (the caller chooses:
     // taking a key/value head's query heads together pays once there are enough (row, key/value head) pairs to fill
     // the GPU; with few rows one block per query head spreads the same work over more blocks).
@@ -468,7 +491,9 @@ TNX_EXPORT int tnx_attention_decode_append(const void* q, int q_stride, void* ca
     if (k_new && (kv_stride % 8 || (((uintptr_t)k_new | (uintptr_t)v_new) & 15))) return TNX_ERR_UNSUPPORTED;
     if (n_splits < 1 || pages_per_split < 1) return TNX_ERR_BAD_ARG;
     if (n_splits > 1 && (!scratch || !counters)) return TNX_ERR_BAD_ARG;
+    if (keep_first < 0 || (bias_mul && !bias_rate)) return TNX_ERR_BAD_ARG;
     DecodeParams p;
+    p.keep_first = keep_first; p.bias.mul = bias_mul; p.bias.rate = bias_rate;
     p.q = (const h16*)q; p.q_stride = q_stride; p.cache = (const h16*)cache;
     p.block_tables = block_tables; p.bt_stride = bt_stride; p.rows = rows; p.token_request = token_request;
     p.positions = positions; p.out = (h16*)out; p.out_stride = out_stride;
@@ -510,7 +535,8 @@ TNX_EXPORT int tnx_attention_decode(const void* q, int q_stride, const void* cac
                                     float* scratch, int* counters, cudaStream_t stream) {
     return tnx_attention_decode_append(q, q_stride, const_cast<void*>(cache), block_tables, bt_stride, rows, token_request,
                                        positions, out, out_stride, n_rows, n_heads, n_kv_heads, head_dim, page_size, window,
-                                       scale, n_splits, pages_per_split, scratch, counters, nullptr, nullptr, 0, 4, 1, stream);
+                                       scale, n_splits, pages_per_split, scratch, counters, nullptr, nullptr, 0, 4, 1, 0, nullptr,
+                                       nullptr, stream);
 }
 
 // ---------------------------------------------------------------------------------------------------

@@ -3,7 +3,7 @@
 //
 // Work item = (request, tile of 128 of its query rows, head).  The queries of a portion sit at
 // positions ctx_len .. ctx_len + q_len - 1 of their request and read the keys 0 .. their own
-// position (or the last `window` of them) from the pages of the request's block table: the keys
+// position (or the last `window` of them, and with a window the first `keep_first`) from the pages of the request's block table: the keys
 // and values of this very portion were written to the pages before the kernel runs.
 //
 // Eight warps, 16 query rows each.  K and V tiles of 64 keys (four pages) are copied to shared
@@ -29,6 +29,8 @@ struct PrefillParams {
     int n_heads, n_kv_heads, head_dim;
     int window;
     float scale_log2;                // scale * log2(e)
+    int keep_first;
+    DistanceBias bias;
 };
 
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -71,7 +73,8 @@ __device__ __forceinline__ uint32_t swz(int row, int chunk) {
     return (uint32_t)(row * (HEAD * 2) + ((chunk ^ (row & 7)) << 4));
 }
 
-template <int HEAD>
+// BIAS: the scores lose a distance bias; they are then carried in log2 units, so that one logarithm a score is all it takes.
+template <int HEAD, bool BIAS>
 __global__ void __launch_bounds__(WARPS * 32, HEAD <= 128 ? 2 : 1)
 attention_prefill_kernel(const PrefillParams p) {
     extern __shared__ __align__(128) uint8_t smem[];
@@ -115,7 +118,12 @@ attention_prefill_kernel(const PrefillParams p) {
     const int r_lo = warp * 16 + (lane >> 2);                // this thread's two rows within the tile
     const int qpos_lo = pos0 + r_lo, qpos_hi = qpos_lo + 8;
 
-    const int key_begin = first_visible_key(pos0, p.window) / BKV * BKV;     // p.window: the mask rule of common.cuh
+    // p.window: the mask rule of common.cuh; tiles of keys are numbered along the walk over the visible ones
+    const BlockWalk walk = walk_blocks(first_visible_key(pos0, p.window), p.keep_first, BKV);
+    const int n_tiles = walk.count(pos_last / BKV);
+    const float scale_log2 = BIAS ? 1.f : p.scale_log2;      // of the scores as they are carried
+    float bias_mul = 0.f, bias_rate = 0.f;
+    if (BIAS) { bias_mul = p.bias.mul[h]; bias_rate = p.bias.rate[h]; }
     const int first_lo = first_visible_key(qpos_lo, p.window), first_hi = first_visible_key(qpos_hi, p.window);
     const size_t head_block = (size_t)PAGE * d;
 
@@ -137,12 +145,12 @@ attention_prefill_kernel(const PrefillParams p) {
         }
         cp_async_commit();
     };
-    load_tile(key_begin, 0);
-    int tile_no = 0;
-    for (int k0 = key_begin; k0 <= pos_last; k0 += BKV, ++tile_no) {
+    load_tile(walk.at(0) * BKV, 0);
+    for (int tile_no = 0; tile_no < n_tiles; ++tile_no) {
+        const int k0 = walk.at(tile_no) * BKV;
         const int buf = tile_no & 1;
-        const bool has_next = k0 + BKV <= pos_last;
-        if (has_next) load_tile(k0 + BKV, buf ^ 1);          // its buffer was released by the barrier below
+        const bool has_next = tile_no + 1 < n_tiles;
+        if (has_next) load_tile(walk.at(tile_no + 1) * BKV, buf ^ 1);          // its buffer was released by the barrier below
         if (has_next) cp_async_wait_one(); else cp_async_wait_all();
         __syncthreads();
         const uint8_t* sK = sKV + (size_t)buf * 2 * KV_BYTES;
@@ -169,12 +177,25 @@ attention_prefill_kernel(const PrefillParams p) {
             }
         }
         // ---- mask, online softmax ------------------------------------------------------------------
+        if constexpr (BIAS) {
+#pragma unroll
+            for (int nt = 0; nt < BKV / 8; ++nt) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int key = k0 + nt * 8 + (lane & 3) * 2 + (e & 1);
+                    // (a key behind the query, masked below, must not make a NaN of the row's maximum)
+                    const float dist = fmaxf((float)(((e < 2) ? qpos_lo : qpos_hi) - key), 0.f);
+                    s[nt][e] = fmaf(s[nt][e], p.scale_log2, -bias_mul * log2_approx(fmaf(bias_rate, dist, 1.f)));
+                }
+            }
+        }
         // The running maximum is kept on the raw scores (the scale is positive); one FMA folds the
         // scale and the maximum into the argument of ex2.  Only tiles that reach past the smallest
         // position of this warp's rows (or fall partly behind the window) need the mask.
         const int warp_pos_lo = pos0 + warp * 16, warp_pos_hi = warp_pos_lo + 15;
         bool need_mask = k0 + BKV - 1 > warp_pos_lo;
-        if (p.window != 0) need_mask = need_mask || k0 < first_visible_key(warp_pos_hi, p.window);
+        if (p.window != 0)
+            need_mask = need_mask || (k0 < first_visible_key(warp_pos_hi, p.window) && k0 + BKV > p.keep_first);
         if (need_mask) {
 #pragma unroll
             for (int nt = 0; nt < BKV / 8; ++nt) {
@@ -182,7 +203,7 @@ attention_prefill_kernel(const PrefillParams p) {
                 for (int e = 0; e < 4; ++e) {
                     const int key = k0 + nt * 8 + (lane & 3) * 2 + (e & 1);
                     const int qp = (e < 2) ? qpos_lo : qpos_hi;
-                    const bool ok = key <= qp && key >= ((e < 2) ? first_lo : first_hi);
+                    const bool ok = key <= qp && (key >= ((e < 2) ? first_lo : first_hi) || key < p.keep_first);
                     if (!ok) s[nt][e] = -INFINITY;
                 }
             }
@@ -199,8 +220,8 @@ attention_prefill_kernel(const PrefillParams p) {
             mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 1));
             mx[r] = fmaxf(mx[r], __shfl_xor_sync(0xffffffffu, mx[r], 2));
             const float m_new = fmaxf(m_run[r], mx[r]);
-            m_scaled[r] = (m_new == -INFINITY) ? 0.f : m_new * p.scale_log2;
-            corr[r] = (m_run[r] == -INFINITY) ? 0.f : ex2_approx(m_run[r] * p.scale_log2 - m_scaled[r]);
+            m_scaled[r] = (m_new == -INFINITY) ? 0.f : m_new * scale_log2;
+            corr[r] = (m_run[r] == -INFINITY) ? 0.f : ex2_approx(m_run[r] * scale_log2 - m_scaled[r]);
             m_run[r] = m_new;
             l_run[r] *= corr[r];
         }
@@ -213,7 +234,7 @@ attention_prefill_kernel(const PrefillParams p) {
         for (int nt = 0; nt < BKV / 8; ++nt) {
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
-                const float pv = ex2_approx(fmaf(s[nt][e], p.scale_log2, -m_scaled[e >> 1]));   // ex2(-inf) = 0
+                const float pv = ex2_approx(fmaf(s[nt][e], scale_log2, -m_scaled[e >> 1]));   // ex2(-inf) = 0
                 s[nt][e] = pv;
                 rs[e >> 1] += pv;
             }
@@ -260,17 +281,22 @@ attention_prefill_kernel(const PrefillParams p) {
     }
 }
 
-template <int HEAD>
-int launch(const PrefillParams& p, int n_items, cudaStream_t stream) {
+template <int HEAD, bool BIAS>
+int launch_as(const PrefillParams& p, int n_items, cudaStream_t stream) {
     constexpr int smem = (BQ + 4 * BKV) * HEAD * 2;
     static bool configured = false;
     if (!configured && smem > 48 * 1024) {
-        cudaError_t e = cudaFuncSetAttribute(attention_prefill_kernel<HEAD>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        cudaError_t e = cudaFuncSetAttribute(attention_prefill_kernel<HEAD, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
     dim3 grid(p.n_heads, n_items);        // heads vary fastest: CTAs start in the order of the work items
-    return tnx_launch_in_order(attention_prefill_kernel<HEAD>, grid, dim3(WARPS * 32), smem, stream, p);
+    return tnx_launch_in_order(attention_prefill_kernel<HEAD, BIAS>, grid, dim3(WARPS * 32), smem, stream, p);
+}
+
+template <int HEAD>
+int launch(const PrefillParams& p, int n_items, cudaStream_t stream) {
+    return p.bias.mul ? launch_as<HEAD, true>(p, n_items, stream) : launch_as<HEAD, false>(p, n_items, stream);
 }
 
 }  // namespace
@@ -279,13 +305,16 @@ TNX_EXPORT int tnx_attention_prefill(const void* q, int q_stride, const void* ca
                                      int bt_stride, const int* tile_req, const int* tile_q0, const int* q_start,
                                      const int* q_len, const int* ctx_len, void* out, int out_stride, int n_items,
                                      int n_heads, int n_kv_heads, int head_dim, int page_size, int window,
-                                     float scale, cudaStream_t stream) {
+                                     float scale, int keep_first, const float* bias_mul, const float* bias_rate,
+                                     cudaStream_t stream) {
     if (n_items <= 0) return 0;
     if (page_size != PAGE || head_dim % 16 || head_dim < 16 || head_dim > 256 || n_kv_heads <= 0 ||
         n_heads % n_kv_heads || q_stride % 8 || out_stride % 2 || ((uintptr_t)q & 15) || ((uintptr_t)cache & 15) ||
         ((uintptr_t)out & 3))
         return TNX_ERR_UNSUPPORTED;
+    if (keep_first < 0 || (bias_mul && !bias_rate)) return TNX_ERR_BAD_ARG;
     PrefillParams p;
+    p.keep_first = keep_first; p.bias.mul = bias_mul; p.bias.rate = bias_rate;
     p.q = (const h16*)q; p.q_stride = q_stride; p.cache = (const h16*)cache; p.block_tables = block_tables;
     p.bt_stride = bt_stride; p.tile_req = tile_req; p.tile_q0 = tile_q0; p.q_start = q_start; p.q_len = q_len;
     p.ctx_len = ctx_len; p.out = (h16*)out; p.out_stride = out_stride; p.n_heads = n_heads; p.n_kv_heads = n_kv_heads;

@@ -59,6 +59,8 @@ struct TcPrefillParams {
     int n_heads, n_kv_heads;
     int window;
     float scale_log2;
+    int keep_first;              // with a window: the first positions that stay visible
+    DistanceBias bias;
     int* err;
 };
 
@@ -106,7 +108,8 @@ __host__ __device__ constexpr uint32_t idesc_attn(int n, int b_mn) {
     return (1u << 4) | IDESC_H16_AB | ((uint32_t)b_mn << 16) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(128 >> 4) << 24);
 }
 
-template <int D, int K_STAGES, int V_STAGES>
+// BIAS: the scores lose a distance bias; they are then carried in log2 units.
+template <int D, int K_STAGES, int V_STAGES, bool BIAS>
 __global__ void __launch_bounds__(THREADS, 2)
 attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_kv,
                             const TcPrefillParams p) {
@@ -145,15 +148,21 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     const int* bt = p.block_tables + (size_t)req * p.bt_stride;
     const int pos0 = ctx + q0, pos_last = pos0 + rows - 1;
     const int kv_total = ctx + ql;
-    const int key_begin = first_visible_key(pos0, p.window) / BKV * BKV;     // p.window: the mask rule of common.cuh
-    const int n_tiles = (pos_last - key_begin) / BKV + 1;
+    // p.window: the mask rule of common.cuh; tiles of keys are numbered along the walk over the visible ones
+    const BlockWalk walk = walk_blocks(first_visible_key(pos0, p.window), p.keep_first, BKV);
+    const int n_tiles = walk.count(pos_last / BKV);
 
     // K and V stages start as zeros: pages that do not exist are not loaded, and what a stage holds
     // then must be finite (it is multiplied by probabilities that are zero).
     for (int i = threadIdx.x; i < (K_STAGES + V_STAGES) * KV_BYTES / 16; i += THREADS) ((uint4*)sK)[i] = make_uint4(0, 0, 0, 0);
-    const int first_page = key_begin / PAGE;
-    const int n_pages = (min(kv_total, key_begin + n_tiles * BKV) - key_begin + PAGE - 1) / PAGE;   // pages that exist
-    for (int i = threadIdx.x; i < n_pages && i < MAX_PAGES_SMEM; i += THREADS) pages_s[i] = bt[first_page + i];
+    // the i-th page of the walk's tiles is block walk.at(i / 4) * 4 + i % 4 of the request; it exists below n_blocks
+    constexpr int TILE_PAGES = BKV / PAGE;
+    const int n_blocks = (kv_total + PAGE - 1) / PAGE;
+    auto page_of = [&](int i) {
+        const int b = walk.at(i / TILE_PAGES) * TILE_PAGES + i % TILE_PAGES;
+        return b < n_blocks ? bt[b] : -1;
+    };
+    for (int i = threadIdx.x; i < n_tiles * TILE_PAGES && i < MAX_PAGES_SMEM; i += THREADS) pages_s[i] = page_of(i);
     if (threadIdx.x == 0) {
         mbar_init(&q_full, 1);
         for (int s = 0; s < K_STAGES; ++s) { mbar_init(&k_full[s], 1); mbar_init(&k_empty[s], 1); }
@@ -186,20 +195,17 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             for (int sl = 0; sl < SLICES; ++sl) tma_load_2d(sQ + sl * ATOM_Q, &map_q, &q_full, h * D + sl * 64, qs + q0);
         }
         const int g = (lane >> 1) & 3, a = lane & 1;          // this lane's page of the tile and half of the head
-        // the page this lane copies for key tile j (-1 where the context ends before), and how many pages exist
-        auto tile_page = [&](int j, int& n_valid) {
-            const int first = j * 4;
-            n_valid = min(4, max(0, n_pages - first));
-            const int i = first + g;
-            return i < n_pages ? (i < MAX_PAGES_SMEM ? pages_s[i] : bt[first_page + i]) : -1;
+        // the page this lane copies for key tile j (-1 where the context ends before)
+        auto tile_page = [&](int j) {
+            const int i = j * TILE_PAGES + g;
+            return i < MAX_PAGES_SMEM ? pages_s[i] : page_of(i);
         };
         auto load_tile = [&](int j, int which, uint8_t* stage, uint64_t* full, uint64_t* empty, uint32_t parity, int code) {
-            int n_valid;
-            const int page = tile_page(j, n_valid);
+            const int page = tile_page(j);
             // Only pages that are copied are announced: behind a sliding window the first tile may
             // begin with blocks that were given back already (-1 in the block table); their part of
             // the stage keeps finite numbers, and the window masks those keys.
-            n_valid = __popc(__ballot_sync(0xffffffffu, lane < 8 && a == 0 && page >= 0));
+            const int n_valid = __popc(__ballot_sync(0xffffffffu, lane < 8 && a == 0 && page >= 0));
             int good = 1;
             if (lane == 0) {
                 good = mbar_wait(empty, parity, p.err, code) ? 1 : 0;
@@ -286,9 +292,12 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const int qpos = pos0 + r;
         const int first_key = first_visible_key(qpos, p.window);
         float m_run = -INFINITY, l_run = 0.f;
+        const float scale_log2 = BIAS ? 1.f : p.scale_log2;      // of the scores as they are carried
+        float bias_mul = 0.f, bias_rate = 0.f;
+        if constexpr (BIAS) { bias_mul = p.bias.mul[h]; bias_rate = p.bias.rate[h]; }
         for (int j = 0; j < n_tiles && ok; ++j) {
             const int b = j & 1;
-            const int k0 = key_begin + j * BKV;
+            const int k0 = walk.at(j) * BKV;
             ok = mbar_wait(&s_full[b], (uint32_t)((j >> 1) & 1), p.err, 37);
             if (!ok) break;
             tc_fence_after();
@@ -303,12 +312,19 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
 #pragma unroll
             for (int i = 0; i < 32; ++i) { s[i] = __uint_as_float(raw0[i]); s[32 + i] = __uint_as_float(raw1[i]); }
             bool need_mask = k0 + BKV - 1 > qpos;
-            need_mask = need_mask || k0 < first_key;
+            need_mask = need_mask || (k0 < first_key && k0 + BKV > p.keep_first);
+            if constexpr (BIAS) {
+                // (a key behind the query, masked below, must not make a NaN of the row's maximum)
+                const float d0 = (float)(qpos - k0);
+#pragma unroll
+                for (int i = 0; i < 64; ++i)
+                    s[i] = fmaf(s[i], p.scale_log2, -bias_mul * log2_approx(fmaf(bias_rate, fmaxf(d0 - (float)i, 0.f), 1.f)));
+            }
             if (need_mask) {
 #pragma unroll
                 for (int i = 0; i < 64; ++i) {
                     const int key = k0 + i;
-                    if (key > qpos || key < first_key) s[i] = -INFINITY;
+                    if (key > qpos || (key < first_key && key >= p.keep_first)) s[i] = -INFINITY;
                 }
             }
             // the row's maximum and sum as four chains each: no instruction waits for the one before it
@@ -320,7 +336,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             // grown by more than 2^RESCALE_STEP: until then P holds values up to 2^RESCALE_STEP
             // instead of 1, which 32-bit sums and bfloat16 products carry as well, and O (which a
             // move of the reference has to rescale in tensor memory) is left alone.
-            const float mx_scaled = (mx == -INFINITY) ? -INFINITY : mx * p.scale_log2;
+            const float mx_scaled = (mx == -INFINITY) ? -INFINITY : mx * scale_log2;
             const bool grow = mx_scaled > m_run + RESCALE_STEP;            // m_run: the reference, in log2 units
             const float m_new = grow ? mx_scaled : m_run;
             const float m_scaled = (m_new == -INFINITY) ? 0.f : m_new;
@@ -329,8 +345,8 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
             uint32_t packed[32];
 #pragma unroll
             for (int i = 0; i < 32; ++i) {
-                const float p0 = ex2_approx(fmaf(s[2 * i], p.scale_log2, -m_scaled));
-                const float p1 = ex2_approx(fmaf(s[2 * i + 1], p.scale_log2, -m_scaled));
+                const float p0 = ex2_approx(fmaf(s[2 * i], scale_log2, -m_scaled));
+                const float p1 = ex2_approx(fmaf(s[2 * i + 1], scale_log2, -m_scaled));
                 sum4[i & 3] += p0 + p1;
                 h16x2 h2 = floats_to_h16x2(p0, p1);
                 packed[i] = *(uint32_t*)&h2;
@@ -404,16 +420,22 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
     }
 }
 
-template <int D, int KS, int VS>
-int launch_tc(const CUtensorMap& mq, const CUtensorMap& mkv, const TcPrefillParams& p, int n_heads, int n_items, cudaStream_t stream) {
+template <int D, int KS, int VS, bool BIAS>
+int launch_tc_as(const CUtensorMap& mq, const CUtensorMap& mkv, const TcPrefillParams& p, int n_heads, int n_items, cudaStream_t stream) {
     constexpr int smem = Layout<D, KS, VS>::SMEM_BYTES;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<D, KS, VS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
+        cudaError_t e = cudaFuncSetAttribute(attention_prefill_tc_kernel<D, KS, VS, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem);
         if (e != cudaSuccess) return (int)e;
         configured = true;
     }
-    return tnx_launch_in_order(attention_prefill_tc_kernel<D, KS, VS>, dim3(n_heads, n_items), dim3(THREADS), smem, stream, mq, mkv, p);   // heads vary fastest
+    return tnx_launch_in_order(attention_prefill_tc_kernel<D, KS, VS, BIAS>, dim3(n_heads, n_items), dim3(THREADS), smem, stream, mq, mkv, p);   // heads vary fastest
+}
+
+template <int D, int KS, int VS>
+int launch_tc(const CUtensorMap& mq, const CUtensorMap& mkv, const TcPrefillParams& p, int n_heads, int n_items, cudaStream_t stream) {
+    return p.bias.mul ? launch_tc_as<D, KS, VS, true>(mq, mkv, p, n_heads, n_items, stream)
+                      : launch_tc_as<D, KS, VS, false>(mq, mkv, p, n_heads, n_items, stream);
 }
 
 }  // namespace
@@ -424,12 +446,14 @@ TNX_EXPORT int tnx_attention_prefill_tc(const void* q, int q_stride, int n_rows_
                                         const int* block_tables, int bt_stride, const int* tile_req, const int* tile_q0,
                                         const int* q_start, const int* q_len, const int* ctx_len, void* out,
                                         int out_stride, int n_items, int n_heads, int n_kv_heads, int head_dim,
-                                        int page_size, int window, float scale, int* err_word, cudaStream_t stream) {
+                                        int page_size, int window, float scale, int keep_first, const float* bias_mul,
+                                        const float* bias_rate, int* err_word, cudaStream_t stream) {
     if (n_items <= 0) return 0;
     if (head_dim < 64 || head_dim > 128 || head_dim % 16 || page_size != PAGE || n_kv_heads <= 0 || n_heads % n_kv_heads || q_stride % 8 ||
         out_stride % 8 || ((uintptr_t)q & 15) || ((uintptr_t)cache & 15) || ((uintptr_t)out & 15) ||
         cache_rows > 0x7fffffffLL || !err_word)
         return TNX_ERR_UNSUPPORTED;
+    if (keep_first < 0 || (bias_mul && !bias_rate)) return TNX_ERR_BAD_ARG;
     CUtensorMap mq, mkv;
     if (!make_map(&mq, q, n_rows_q, n_heads * head_dim, q_stride, BQ)) return TNX_ERR_UNSUPPORTED;
     if (!make_map(&mkv, cache, (int)cache_rows, head_dim, head_dim, PAGE)) return TNX_ERR_UNSUPPORTED;
@@ -437,7 +461,7 @@ TNX_EXPORT int tnx_attention_prefill_tc(const void* q, int q_stride, int n_rows_
     p.block_tables = block_tables; p.bt_stride = bt_stride; p.tile_req = tile_req; p.tile_q0 = tile_q0;
     p.q_start = q_start; p.q_len = q_len; p.ctx_len = ctx_len; p.out = (h16*)out; p.out_stride = out_stride;
     p.n_heads = n_heads; p.n_kv_heads = n_kv_heads; p.window = window; p.scale_log2 = scale * 1.4426950408889634f;
-    p.err = err_word;
+    p.err = err_word; p.keep_first = keep_first; p.bias.mul = bias_mul; p.bias.rate = bias_rate;
     switch (head_dim) {
         case 128: return launch_tc<128, 2, 3>(mq, mkv, p, n_heads, n_items, stream);
         case 112: return launch_tc<112, 2, 3>(mq, mkv, p, n_heads, n_items, stream);

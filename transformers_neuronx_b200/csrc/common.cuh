@@ -177,6 +177,35 @@ __host__ __device__ __forceinline__ int first_visible_key(int pos, int mask) {
     return 0;
 }
 
+// With a sliding window the first `keep` positions may stay visible to every later query (keep 0: not): a query at `pos`
+// then reads key j <= pos where j >= first_visible_key(pos, mask) or j < keep.  A kernel that walks the keys in blocks of
+// a fixed size takes the blocks of the first positions, then jumps to the block of the first key behind the gap.
+struct BlockWalk {
+    int kept, first;             // blocks 0 .. kept - 1, then first, first + 1, ...
+    __host__ __device__ __forceinline__ int at(int i) const { return i < kept ? i : first + i - kept; }
+    // how many blocks lie on the walk up to and with block `last` (last >= first), and the place of block b >= first on it
+    __host__ __device__ __forceinline__ int count(int last) const { return kept + last - first + 1; }
+    __host__ __device__ __forceinline__ int place(int b) const { return kept + b - first; }
+};
+__host__ __device__ __forceinline__ BlockWalk walk_blocks(int first_key, int keep, int block) {
+    const int fb = first_key / block, kb = keep > 0 ? (keep + block - 1) / block : 0;
+    BlockWalk w;
+    if (keep > 0 && kb >= fb) { w.kept = 0; w.first = 0; }        // no block between them: all from the start
+    else { w.kept = kb; w.first = fb; }
+    return w;
+}
+
+// A distance bias that is taken off the scores of head h: mul[h] * ln(1 + rate[h] * (i - j)) (mul null: none).
+struct DistanceBias {
+    const float* mul;
+    const float* rate;
+};
+__device__ __forceinline__ float log2_approx(float x) {
+    float y;
+    asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

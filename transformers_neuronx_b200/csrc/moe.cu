@@ -1,6 +1,6 @@
 // A feed-forward of routed experts.
 //
-//   z = W_r h                                  router logits, 32-bit sums
+//   z = W_r h (+ bias)                         router logits, 32-bit sums
 //   s = sigmoid(z) (or softmax(z))             scores; the `top` largest choose the token's experts
 //   w_j = s[e_j] (optionally divided by their sum)
 //   expert e on input x:  g = W_gate x, u = W_up x (both clamped where the part gives limits),
@@ -78,6 +78,7 @@ struct RouterOptions {
     const float* correction;     // [E] or null
     int n_groups, keep_groups, group_top;
     float renorm_eps, weight_scale;
+    const float* bias;           // [E], added to the logits, or null
 };
 
 template <typename T, typename TW>
@@ -102,7 +103,7 @@ moe_router_kernel(const T* __restrict__ h, int ld, const TW* __restrict__ wr, co
     const bool vec = W % 8 == 0 && ((uintptr_t)wr % 16) == 0;
     for (int e = warp; e < E; e += 4) {
         const float s = warp_dot<TW>(wr + (size_t)e * W, x, W, lane, vec);
-        if (lane == 0) z[e] = s;
+        if (lane == 0) z[e] = s + (ro.bias ? ro.bias[e] : 0.f);
     }
     __syncthreads();
     if (warp != 0) return;
@@ -431,14 +432,14 @@ moe_sum_kernel(const float* __restrict__ per_pair, const int* __restrict__ ids, 
 TNX_EXPORT int tnx_moe_route(const void* h, int ld, const void* router, const int* token_request, int* ids, float* weights,
                              int N, int W, int E, int top, int softmax_scores, int renormalize, int h_h16, int w_h16,
                              const float* correction, int n_groups, int keep_groups, int group_top, float renorm_eps,
-                             float weight_scale, cudaStream_t stream) {
+                             float weight_scale, const float* bias, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (W <= 0 || E <= 0 || E > MAX_EXPERTS || top <= 0 || top > MAX_TOP || top > E) return TNX_ERR_UNSUPPORTED;
     if (n_groups < 1 || E % n_groups || keep_groups < 1 || keep_groups > n_groups || group_top < 1 ||
         (long long)keep_groups * (E / n_groups) < top || ((correction || n_groups > 1) && softmax_scores))
         return TNX_ERR_BAD_ARG;
     if (n_groups > 1 && E / n_groups > 64 && group_top > 1) return TNX_ERR_UNSUPPORTED;
-    const RouterOptions ro{correction, n_groups, keep_groups, group_top, renorm_eps, weight_scale};
+    const RouterOptions ro{correction, n_groups, keep_groups, group_top, renorm_eps, weight_scale, bias};
     const size_t smem = (size_t)(((W + 3) & ~3) + 3 * E) * sizeof(float);
     if (smem > 160 * 1024) return TNX_ERR_UNSUPPORTED;
 #define GO(T, TW)                                                                                                       \

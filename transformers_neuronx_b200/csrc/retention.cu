@@ -5,9 +5,9 @@
 // Everything that enters the recurrence is 32-bit: queries and keys are rotated by position in 32-bit from the
 // projection's output (tnx_retention_prep) and are not rounded again; the state lives in 32-bit.
 //
-// tnx_retention_prep: on the first rot_dims dims of each head, dim i paired with i + rot_dims/2, the pair
+// tnx_retention_prep: queries, keys and (where asked for) values pass an activation; then on the first rot_dims dims of each head, dim i paired with i + rot_dims/2, the pair
 //   (u, v) at position p becomes (u cos a - v sin a, v cos a + u sin a), a = p * inv_freq[i]; keys are then
-//   multiplied by k_scale.  Output: 32-bit q and k, [tokens, heads * k_dim].
+//   multiplied by k_scale.  Output: 32-bit q and k, [tokens, heads * k_dim] (and 32-bit values).
 // tnx_retention_scan: a thread block owns C columns (value dims) of one head of one request and walks the
 //   request's tokens of this step in order, the state's columns in registers: a column's k_dim rows are spread
 //   over R adjacent lanes, which add their partial sums of o_t with shuffles.  The state is stored
@@ -16,7 +16,7 @@
 //   keeps it in registers for all its tokens.  Queries and keys of a few tokens at a time are staged in shared memory.
 // tnx_headwise_gated_rms_norm: o of each (token, head) divided by its root mean square (eps inside the root,
 //   an optional weight over the head's dims), multiplied by act(gate) (silu here; the activation is a parameter) and
-//   by out_scale, written in the activation type.
+//   by out_scale, written in the activation type.  tnx_gated_rms_norm: the same over all heads of a token together.
 #include "common.cuh"
 
 namespace {
@@ -25,7 +25,8 @@ template <typename T>
 __global__ void retention_prep_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off,
                                       const int* __restrict__ token_request, const int* __restrict__ positions,
                                       const float* __restrict__ inv_freq, int rot_dims, float k_scale,
-                                      float* __restrict__ q_out, float* __restrict__ k_out, int H, int dk) {
+                                      float* __restrict__ q_out, float* __restrict__ k_out, int H, int dk, int act, int v_off,
+                                      float* __restrict__ v_out, int nv) {
     extern __shared__ float sm[];                   // cos and sin of the token's angles, the same for every head
     pdl_launch_dependents();
     pdl_wait();
@@ -44,8 +45,8 @@ __global__ void retention_prep_kernel(const T* __restrict__ proj, int ld, int q_
         const int h = e / half, i = e % half;
         const int c0 = h * dk + i, c1 = c0 + half;
         const float sn = snt[i], cs = cst[i];
-        const float qu = to_float(row[q_off + c0]), qv = to_float(row[q_off + c1]);
-        const float ku = to_float(row[k_off + c0]), kv = to_float(row[k_off + c1]);
+        const float qu = apply_activation(to_float(row[q_off + c0]), act), qv = apply_activation(to_float(row[q_off + c1]), act);
+        const float ku = apply_activation(to_float(row[k_off + c0]), act), kv = apply_activation(to_float(row[k_off + c1]), act);
         qd[c0] = qu * cs - qv * sn;
         qd[c1] = qv * cs + qu * sn;
         kd[c0] = (ku * cs - kv * sn) * k_scale;
@@ -54,8 +55,37 @@ __global__ void retention_prep_kernel(const T* __restrict__ proj, int ld, int q_
     const int rest = dk - rot_dims;
     for (int e = threadIdx.x; e < H * rest; e += blockDim.x) {
         const int c = (e / rest) * dk + rot_dims + e % rest;
-        qd[c] = to_float(row[q_off + c]);
-        kd[c] = to_float(row[k_off + c]) * k_scale;
+        qd[c] = apply_activation(to_float(row[q_off + c]), act);
+        kd[c] = apply_activation(to_float(row[k_off + c]), act) * k_scale;
+    }
+    if (v_out)
+        for (int c = threadIdx.x; c < nv; c += blockDim.x) v_out[(size_t)n * nv + c] = apply_activation(to_float(row[v_off + c]), act);
+}
+
+// The same without a rotation, eight neighbouring columns a thread (16-byte loads; sizes and addresses in multiples of eight).
+template <typename T>
+__global__ void retention_prep_vec_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off,
+                                          const int* __restrict__ token_request, float k_scale, float* __restrict__ q_out,
+                                          float* __restrict__ k_out, int nq, int act, int v_off, float* __restrict__ v_out, int nv) {
+    pdl_launch_dependents();
+    pdl_wait();
+    const int n = blockIdx.x;
+    if (token_request[n] < 0) return;
+    const T* row = proj + (size_t)n * ld;
+    const int all = 2 * nq + nv;
+    for (int e = 8 * (blockIdx.y * blockDim.x + threadIdx.x); e < all; e += 8 * gridDim.y * blockDim.x) {
+        const int which = e < nq ? 0 : (e < 2 * nq ? 1 : 2), c = e - which * nq;
+        Vec8<T> raw;
+        raw.load(row + (which == 0 ? q_off : (which == 1 ? k_off : v_off)) + c);
+        float f[8];
+        raw.get(f);
+        const float scale = which == 1 ? k_scale : 1.f;
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] = apply_activation(f[i], act) * scale;
+        float* dst = which == 0 ? q_out + (size_t)n * nq + c : (which == 1 ? k_out + (size_t)n * nq + c : v_out + (size_t)n * nv + c);
+        Vec8<float> o;
+        o.set(f);
+        o.store(dst);
     }
 }
 
@@ -382,7 +412,7 @@ retention_decode_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off
                         float k_scale, const float* __restrict__ decay, float* __restrict__ state,
                         const int* __restrict__ q_start, const int* __restrict__ q_len,
                         const int* __restrict__ state_slots, float eps, float out_scale, T* __restrict__ out, int out_ld,
-                        int H, int dk, int dv) {
+                        int H, int dk, int dv, int act, int gate_act, float* __restrict__ raw_out) {
     constexpr int DKP = KPT * R;
     constexpr int GROUP = 4 * R + 4;
     extern __shared__ __align__(16) float sm[];      // q [DKP], k [DKP], v [dv4], gate [dv4], part [CG][GROUP], o [dv4]
@@ -408,14 +438,15 @@ retention_decode_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off
         float qv = 0.f, kv = 0.f;
         if (i < dk) {
             const int c = h * dk + i;
-            qv = to_float(row[q_off + c]);
-            kv = to_float(row[k_off + c]);
+            qv = apply_activation(to_float(row[q_off + c]), act);
+            kv = apply_activation(to_float(row[k_off + c]), act);
             if (i < rot_dims) {
                 const int fi = i < half ? i : i - half;
                 float sn, cs;
                 sincosf(pos * inv_freq[fi], &sn, &cs);
                 const int partner = i < half ? c + half : c - half;
-                const float q2 = to_float(row[q_off + partner]), k2 = to_float(row[k_off + partner]);
+                const float q2 = apply_activation(to_float(row[q_off + partner]), act);
+                const float k2 = apply_activation(to_float(row[k_off + partner]), act);
                 // the pair (u, v) becomes (u cos - v sin, v cos + u sin)
                 qv = i < half ? qv * cs - q2 * sn : qv * cs + q2 * sn;
                 kv = i < half ? kv * cs - k2 * sn : kv * cs + k2 * sn;
@@ -426,7 +457,7 @@ retention_decode_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off
         ks[i] = kv;
     }
     for (int j = threadIdx.x; j < dv4; j += blockDim.x) {
-        vs[j] = j < dv ? to_float(row[v_off + h * dv + j]) : 0.f;
+        vs[j] = j < dv ? apply_activation(to_float(row[v_off + h * dv + j]), act) : 0.f;
         gs[j] = (j < dv && g_off >= 0) ? to_float(row[g_off + h * dv + j]) : 0.f;
     }
     __syncthreads();
@@ -478,13 +509,15 @@ retention_decode_kernel(const T* __restrict__ proj, int ld, int q_off, int k_off
         for (int i = 0; i < R; ++i) a += p[4 * i];
         os[j] = a;
         ss += a * a;
+        if (raw_out) raw_out[(size_t)n * out_ld + (size_t)h * dv + j] = a;
     }
+    if (raw_out) return;
     ss = block_sum(ss, scratch);
     const float rinv = 1.0f / sqrtf(ss / (float)dv + eps);
     T* dst = out + (size_t)n * out_ld + (size_t)h * dv;
     for (int j = threadIdx.x; j < dv; j += blockDim.x) {
         float y = os[j] * rinv;
-        if (g_off >= 0) { const float z = gs[j]; y *= z / (1.f + expf(-z)); }
+        if (g_off >= 0) y *= apply_activation(gs[j], gate_act);
         dst[j] = from_float<T>(y * out_scale);
     }
 }
@@ -542,20 +575,100 @@ __global__ void headwise_gated_rms_norm_kernel(const float* __restrict__ o, cons
     }
 }
 
+// o of a token divided by the root mean square of its whole row (all heads together), times a weight, times
+// act(gate), times out_scale.  A block a token; VEC: runs of eight.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256)
+gated_rms_norm_kernel(const float* __restrict__ o, const T* __restrict__ gate, int gate_ld, const int* __restrict__ token_request,
+                      const float* __restrict__ w, float eps, float out_scale, T* __restrict__ out, int out_ld, int width,
+                      int gate_act) {
+    __shared__ float scratch[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    const int n = blockIdx.x;
+    if (token_request[n] < 0) return;
+    const float* src = o + (size_t)n * width;
+    const T* g = gate ? gate + (size_t)n * gate_ld : nullptr;
+    T* dst = out + (size_t)n * out_ld;
+    float s = 0.f;
+    if constexpr (VEC) {
+        for (int c = 8 * threadIdx.x; c < width; c += 8 * blockDim.x) {
+            Vec8<float> v;
+            v.load(src + c);
+            s += (v.a.x * v.a.x + v.a.y * v.a.y) + (v.a.z * v.a.z + v.a.w * v.a.w);
+            s += (v.b.x * v.b.x + v.b.y * v.b.y) + (v.b.z * v.b.z + v.b.w * v.b.w);
+        }
+    } else {
+        for (int c = threadIdx.x; c < width; c += blockDim.x) s += src[c] * src[c];
+    }
+    const float rinv = 1.0f / sqrtf(block_sum(s, scratch) / (float)width + eps);
+    if constexpr (VEC) {
+        for (int c = 8 * threadIdx.x; c < width; c += 8 * blockDim.x) {
+            Vec8<float> v;
+            float y[8];
+            v.load(src + c);                      // the first-level cache still holds the row
+            v.get(y);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) y[i] *= rinv * out_scale;
+            if (w) {
+                Vec8<float> wv;
+                float f[8];
+                wv.load(w + c);
+                wv.get(f);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) y[i] *= f[i];
+            }
+            if (g) {
+                Vec8<T> gv;
+                float z[8];
+                gv.load(g + c);
+                gv.get(z);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) y[i] *= apply_activation(z[i], gate_act);
+            }
+            Vec8<T> r;
+            r.set(y);
+            r.store(dst + c);
+        }
+    } else {
+        for (int c = threadIdx.x; c < width; c += blockDim.x) {
+            float y = src[c] * rinv * out_scale;
+            if (w) y *= w[c];
+            if (g) y *= apply_activation(to_float(g[c]), gate_act);
+            dst[c] = from_float<T>(y);
+        }
+    }
+}
+
 }  // namespace
 
 TNX_EXPORT int tnx_retention_prep(const void* proj, int ld, int q_off, int k_off, const int* token_request,
                                   const int* positions, const float* inv_freq, int rot_dims, float k_scale, float* q_out,
-                                  float* k_out, int n_tokens, int H, int dk, int is_h16, cudaStream_t stream) {
+                                  float* k_out, int n_tokens, int H, int dk, int act, int v_off, float* v_out, int nv, int is_h16,
+                                  cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
+    if (act < 0 || act >= TNX_ACT_COUNT || nv < 0) return TNX_ERR_BAD_ARG;
     if (H <= 0 || dk <= 0 || rot_dims < 0 || rot_dims > dk || rot_dims % 2 || (rot_dims && !inv_freq)) return TNX_ERR_BAD_ARG;
     const int threads = H * dk >= 2048 ? 256 : 128;
+    const int nq = H * dk;
+    if (!v_out) nv = 0;
+    if (!rot_dims && nq % 8 == 0 && nv % 8 == 0 && ld % 8 == 0 && q_off % 8 == 0 && k_off % 8 == 0 && v_off % 8 == 0 &&
+        !(((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)k_out | (uintptr_t)v_out) & 15)) {
+        const int pieces = (2 * nq + nv) / 8;
+        const int t = pieces >= 256 ? 256 : 128;
+        const dim3 grid(n_tokens, n_tokens < 64 ? (pieces + t - 1) / t : 1);
+        if (is_h16)
+            return tnx_launch_in_order(retention_prep_vec_kernel<h16>, grid, dim3(t), 0, stream, (const h16*)proj, ld, q_off, k_off,
+                                       token_request, k_scale, q_out, k_out, nq, act, v_off, v_out, nv);
+        return tnx_launch_in_order(retention_prep_vec_kernel<float>, grid, dim3(t), 0, stream, (const float*)proj, ld, q_off, k_off,
+                                   token_request, k_scale, q_out, k_out, nq, act, v_off, v_out, nv);
+    }
     const size_t smem = (size_t)rot_dims * sizeof(float);
     if (is_h16)
         return tnx_launch_in_order(retention_prep_kernel<h16>, dim3(n_tokens), dim3(threads), smem, stream, (const h16*)proj, ld,
-                                   q_off, k_off, token_request, positions, inv_freq, rot_dims, k_scale, q_out, k_out, H, dk);
+                                   q_off, k_off, token_request, positions, inv_freq, rot_dims, k_scale, q_out, k_out, H, dk, act, v_off, v_out, nv);
     return tnx_launch_in_order(retention_prep_kernel<float>, dim3(n_tokens), dim3(threads), smem, stream, (const float*)proj, ld,
-                               q_off, k_off, token_request, positions, inv_freq, rot_dims, k_scale, q_out, k_out, H, dk);
+                               q_off, k_off, token_request, positions, inv_freq, rot_dims, k_scale, q_out, k_out, H, dk, act, v_off, v_out, nv);
 }
 
 // The columns a thread block of the scan owns: 16 (8 where the head has fewer; columns beyond the head are
@@ -692,7 +805,8 @@ template <typename T>
 static int retention_decode_launch(const T* proj, int ld, int q_off, int k_off, int v_off, int g_off, const int* positions,
                                    const float* inv_freq, int rot_dims, float k_scale, const float* decay, float* state,
                                    const int* q_start, const int* q_len, const int* state_slots, float eps, float out_scale,
-                                   T* out, int out_ld, int n_requests, int H, int dk, int dv, cudaStream_t stream) {
+                                   T* out, int out_ld, int n_requests, int H, int dk, int dv, int act, int gate_act,
+                                   float* raw_out, cudaStream_t stream) {
     const int CG = (dv + 3) / 4;
 #define RDEC(KPT, R)                                                                                                    \
     do {                                                                                                                \
@@ -702,7 +816,8 @@ static int retention_decode_launch(const T* proj, int ld, int q_off, int k_off, 
         if (smem > 48 * 1024) return TNX_ERR_UNSUPPORTED;                                                               \
         return tnx_launch_in_order(retention_decode_kernel<T, KPT, R>, dim3(H, n_requests), dim3(threads), smem, stream, \
                                    proj, ld, q_off, k_off, v_off, g_off, positions, inv_freq, rot_dims, k_scale, decay, \
-                                   state, q_start, q_len, state_slots, eps, out_scale, out, out_ld, H, dk, dv);         \
+                                   state, q_start, q_len, state_slots, eps, out_scale, out, out_ld, H, dk, dv, act,     \
+                                   gate_act, raw_out);                                                                  \
     } while (0)
     if (dk <= 16) RDEC(4, 4);
     if (dk <= 32) RDEC(4, 8);
@@ -717,8 +832,12 @@ TNX_EXPORT int tnx_retention_decode(const void* proj, int ld, int q_off, int k_o
                                     const int* positions, const float* inv_freq, int rot_dims, float k_scale,
                                     const float* decay, float* state, const int* q_start, const int* q_len,
                                     const int* state_slots, float eps, float out_scale, void* out, int out_ld,
-                                    int n_requests, int H, int dk, int dv, int is_h16, cudaStream_t stream) {
+                                    int n_requests, int H, int dk, int dv, int act, int gate_act, int raw, int is_h16,
+                                    cudaStream_t stream) {
+    // raw: `out` holds floats and receives the recurrence's output as it is
     if (n_requests <= 0) return 0;
+    if (act < 0 || act >= TNX_ACT_COUNT || gate_act < 0 || gate_act >= TNX_ACT_COUNT) return TNX_ERR_BAD_ARG;
+    float* raw_out = raw ? (float*)out : nullptr;
     if (H <= 0 || dk <= 0 || dv <= 0 || H > 65535 || n_requests > 65535 || rot_dims < 0 || rot_dims > dk || rot_dims % 2 ||
         (rot_dims && !inv_freq) || out_ld < H * dv)
         return TNX_ERR_BAD_ARG;
@@ -726,8 +845,28 @@ TNX_EXPORT int tnx_retention_decode(const void* proj, int ld, int q_off, int k_o
     if (is_h16)
         return retention_decode_launch<h16>((const h16*)proj, ld, q_off, k_off, v_off, g_off, positions, inv_freq, rot_dims,
                                             k_scale, decay, state, q_start, q_len, state_slots, eps, out_scale, (h16*)out,
-                                            out_ld, n_requests, H, dk, dv, stream);
+                                            out_ld, n_requests, H, dk, dv, act, gate_act, raw_out, stream);
     return retention_decode_launch<float>((const float*)proj, ld, q_off, k_off, v_off, g_off, positions, inv_freq, rot_dims,
                                           k_scale, decay, state, q_start, q_len, state_slots, eps, out_scale, (float*)out,
-                                          out_ld, n_requests, H, dk, dv, stream);
+                                          out_ld, n_requests, H, dk, dv, act, gate_act, raw_out, stream);
+}
+
+TNX_EXPORT int tnx_gated_rms_norm(const float* o, const void* gate, int gate_ld, const int* token_request, const float* w,
+                                  float eps, float out_scale, void* out, int out_ld, int n_tokens, int width, int gate_act,
+                                  int is_h16, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (width <= 0 || out_ld < width || (gate && gate_ld < width) || gate_act < 0 || gate_act >= TNX_ACT_COUNT) return TNX_ERR_BAD_ARG;
+    const bool vec = width % 8 == 0 && out_ld % 8 == 0 && (!gate || gate_ld % 8 == 0) &&
+                     !(((uintptr_t)o | (uintptr_t)gate | (uintptr_t)w | (uintptr_t)out) & 15);
+    const int threads = width >= 2048 ? 256 : 128;
+#define GRN(T, V)                                                                                                       \
+    return tnx_launch_in_order(gated_rms_norm_kernel<T, V>, dim3(n_tokens), dim3(threads), 0, stream, o, (const T*)gate, \
+                               gate_ld, token_request, w, eps, out_scale, (T*)out, out_ld, width, gate_act)
+    if (is_h16) {
+        if (vec) GRN(h16, true);
+        GRN(h16, false);
+    }
+    if (vec) GRN(float, true);
+    GRN(float, false);
+#undef GRN
 }

@@ -8,13 +8,15 @@
 //   on the first `rot_dims` dims of each head of q and k, dim i paired with dim i + rot_dims/2:
 //       (u, v) <- (u cos a - v sin a, v cos a + u sin a),  a = p * inv_freq_qk[i]
 //   q of head h <- q * head_scale[h]                (skipped without head_scale)
+//   values, when `other` is given: v <- (1 - w) v + w other, w one number (values mixed with another layer's)
 //   values, when inv_freq_v is given: over all v_dim dims, dim m paired with m + v_dim/2, a = p * inv_freq_v[m]
 //   q, k and v are written with `D` dims a head (D >= k_dim, v_dim; the rest zero), the layout the paged
 //   attention kernels take: zeros in q and k leave the scores alone, zeros in v give zero output columns.
 //
 // tnx_rotary_unrotate, one thread block per token at position p: each head's first v_dim output dims of the
-// attention (D a head) are turned back, pair m by -p * inv_freq_v[m], multiplied by out_scale and written
-// v_dim a head into a (possibly wider) activation buffer.
+// attention (D a head) are turned back, pair m by -p * inv_freq_v[m] (or, without inv_freq_v, multiplied by the sigmoid
+// of a gate, one number per head or per dim, where one is given), multiplied by out_scale and written v_dim a head
+// into a (possibly wider) activation buffer.
 #include "common.cuh"
 #pragma nv_diag_suppress 128      // the plain loops behind a vectorised branch that returns are unreachable in that instantiation
 
@@ -42,7 +44,8 @@ __global__ void rotary_qkv_prep_kernel(const T* __restrict__ proj, int ld, int q
                                        const float* __restrict__ wq, const float* __restrict__ wk, float eps,
                                        const float* __restrict__ head_scale, const float* __restrict__ inv_freq_qk,
                                        int rot_dims, const float* __restrict__ inv_freq_v, T* __restrict__ q_out,
-                                       T* __restrict__ k_out, T* __restrict__ v_out, int H, int G, int dk, int dv, int D) {
+                                       T* __restrict__ k_out, T* __restrict__ v_out, int H, int G, int dk, int dv, int D,
+                                       const T* __restrict__ other, int other_ld, const float* __restrict__ mix) {
     extern __shared__ float sm[];                   // q [H * dk], k [G * dk], v [G * dv], then cos/sin of the token's angles
     __shared__ float scratch[32];
     pdl_launch_dependents();
@@ -63,6 +66,8 @@ __global__ void rotary_qkv_prep_kernel(const T* __restrict__ proj, int ld, int q
     float* sn_v = cs_v + hv;
     for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(pos * inv_freq_qk[i], &sn_qk[i], &cs_qk[i]);
     for (int i = threadIdx.x; i < hv; i += blockDim.x) sincosf(pos * inv_freq_v[i], &sn_v[i], &cs_v[i]);
+    const T* orow = other ? other + (size_t)n * other_ld : nullptr;
+    const float wm = other ? mix[0] : 0.f;
     float sq = 0.f, sk = 0.f;
     if constexpr (VEC8) {
         for (int c = threadIdx.x; c < (nq + nk + nv) / 8; c += blockDim.x) {
@@ -70,6 +75,12 @@ __global__ void rotary_qkv_prep_kernel(const T* __restrict__ proj, int ld, int q
             const int col = e < nq ? q_off + e : (e < nq + nk ? k_off + e - nq : v_off + e - nq - nk);
             float f[8];
             unpack8(*(const uint4*)(row + col), f);
+            if (orow && e >= nq + nk) {
+                float o[8];
+                unpack8(*(const uint4*)(orow + e - nq - nk), o);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) f[i] = fmaf(wm, o[i], (1.f - wm) * f[i]);
+            }
             float ss = 0.f;
 #pragma unroll
             for (int i = 0; i < 8; ++i) { qs[e + i] = f[i]; ss += f[i] * f[i]; }
@@ -78,7 +89,11 @@ __global__ void rotary_qkv_prep_kernel(const T* __restrict__ proj, int ld, int q
     } else {
         for (int c = threadIdx.x; c < nq; c += blockDim.x) { const float v = to_float(row[q_off + c]); qs[c] = v; sq += v * v; }
         for (int c = threadIdx.x; c < nk; c += blockDim.x) { const float v = to_float(row[k_off + c]); ks[c] = v; sk += v * v; }
-        for (int c = threadIdx.x; c < nv; c += blockDim.x) vs[c] = to_float(row[v_off + c]);
+        for (int c = threadIdx.x; c < nv; c += blockDim.x) {
+            float v = to_float(row[v_off + c]);
+            if (orow) v = fmaf(wm, to_float(orow[c]), (1.f - wm) * v);
+            vs[c] = v;
+        }
     }
     sq = block_sum(sq, scratch);
     sk = block_sum(sk, scratch);                    // block_sum synchronises: the rows are in shared memory now
@@ -195,7 +210,8 @@ __global__ void rotary_qkv_prep_kernel(const T* __restrict__ proj, int ld, int q
 template <typename T, bool VEC8>
 __global__ void rotary_unrotate_kernel(const T* __restrict__ att, const int* __restrict__ token_request,
                                        const int* __restrict__ positions, const float* __restrict__ inv_freq_v,
-                                       float out_scale, T* __restrict__ out, int out_ld, int H, int dv, int D) {
+                                       float out_scale, T* __restrict__ out, int out_ld, int H, int dv, int D,
+                                       const T* __restrict__ gate, int gate_ld, int gate_per_head) {
     extern __shared__ float sm[];                   // cos and sin of the token's angles, the same for every head
     pdl_launch_dependents();
     pdl_wait();
@@ -235,8 +251,35 @@ __global__ void rotary_unrotate_kernel(const T* __restrict__ att, const int* __r
             dst[h * dv + m + hv] = from_float<T>((v * cs - u * sn) * out_scale);
         }
     } else {
-        for (int e = threadIdx.x; e < H * dv; e += blockDim.x)
-            dst[e] = from_float<T>(to_float(src[(e / dv) * D + e % dv]) * out_scale);
+        const T* g = gate ? gate + (size_t)n * gate_ld : nullptr;
+        if constexpr (VEC8) {
+            const int d8 = dv / 8;
+            for (int e = threadIdx.x; e < H * d8; e += blockDim.x) {
+                const int h = e / d8, m0 = (e % d8) * 8;
+                float u[8];
+                unpack8(*(const uint4*)(src + h * D + m0), u);
+                if (g && gate_per_head) {
+                    const float f = out_scale / (1.f + expf(-to_float(g[h])));
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) u[i] *= f;
+                } else if (g) {
+                    float z[8];
+                    unpack8(*(const uint4*)(g + 8 * e), z);
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) u[i] *= out_scale / (1.f + expf(-z[i]));
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 8; ++i) u[i] *= out_scale;
+                }
+                *(uint4*)(dst + 8 * e) = pack8(u);
+            }
+            return;
+        }
+        for (int e = threadIdx.x; e < H * dv; e += blockDim.x) {
+            float f = out_scale;
+            if (g) f /= 1.f + expf(-to_float(g[gate_per_head ? e / dv : e]));
+            dst[e] = from_float<T>(to_float(src[(e / dv) * D + e % dv]) * f);
+        }
     }
 }
 
@@ -246,8 +289,10 @@ TNX_EXPORT int tnx_rotary_qkv_prep(const void* proj, int ld, int q_off, int k_of
                                    const int* positions, const float* wq, const float* wk, float eps,
                                    const float* head_scale, const float* inv_freq_qk, int rot_dims,
                                    const float* inv_freq_v, void* q_out, void* k_out, void* v_out, int n_tokens, int H,
-                                   int G, int dk, int dv, int D, int is_h16, cudaStream_t stream) {
+                                   int G, int dk, int dv, int D, const void* other, int other_ld, const float* mix, int is_h16,
+                                   cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
+    if (other && (!mix || inv_freq_v || other_ld < G * dv)) return TNX_ERR_BAD_ARG;
     if (H <= 0 || G <= 0 || dk <= 0 || dv <= 0 || D < dk || D < dv || rot_dims < 0 || rot_dims > dk || rot_dims % 2 ||
         (rot_dims && !inv_freq_qk) || (inv_freq_v && dv % 2))
         return TNX_ERR_BAD_ARG;
@@ -261,11 +306,11 @@ TNX_EXPORT int tnx_rotary_qkv_prep(const void* proj, int ld, int q_off, int k_of
         return tnx_launch_in_order(rotary_qkv_prep_kernel<T, V8>, dim3(n_tokens), dim3(threads), smem, stream,          \
                                    (const T*)proj, ld, q_off, k_off, v_off, token_request, positions, wq, wk, eps,      \
                                    head_scale, inv_freq_qk, rot_dims, inv_freq_v, (T*)q_out, (T*)k_out, (T*)v_out, H,   \
-                                   G, dk, dv, D);                                                                       \
+                                   G, dk, dv, D, (const T*)other, other_ld, mix);                                       \
     } while (0)
     const bool v8 = is_h16 && dk % 8 == 0 && dv % 8 == 0 && D % 8 == 0 && rot_dims % 16 == 0 && (!inv_freq_v || dv % 16 == 0) &&
                     ld % 8 == 0 && q_off % 8 == 0 && k_off % 8 == 0 && v_off % 8 == 0 && ((uintptr_t)proj % 16) == 0 &&
-                    ((uintptr_t)q_out % 16) == 0 && ((uintptr_t)k_out % 16) == 0 && ((uintptr_t)v_out % 16) == 0;
+                    ((uintptr_t)q_out % 16) == 0 && ((uintptr_t)k_out % 16) == 0 && ((uintptr_t)v_out % 16) == 0 && ((uintptr_t)other % 16) == 0 && other_ld % 8 == 0;
     if (is_h16 && v8) PREP_LAUNCH(h16, true);
     if (is_h16) PREP_LAUNCH(h16, false);
     PREP_LAUNCH(float, false);
@@ -274,20 +319,25 @@ TNX_EXPORT int tnx_rotary_qkv_prep(const void* proj, int ld, int q_off, int k_of
 
 TNX_EXPORT int tnx_rotary_unrotate(const void* att, const int* token_request, const int* positions,
                                    const float* inv_freq_v, float out_scale, void* out, int out_ld, int n_tokens, int H,
-                                   int dv, int D, int is_h16, cudaStream_t stream) {
+                                   int dv, int D, const void* gate, int gate_ld, int gate_per_head, int is_h16,
+                                   cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
+    if (gate && (inv_freq_v || gate_ld < (gate_per_head ? H : H * dv))) return TNX_ERR_BAD_ARG;
     if (H <= 0 || dv <= 0 || D < dv || (inv_freq_v && dv % 2) || out_ld < H * dv) return TNX_ERR_BAD_ARG;
     const int threads = H * dv >= 2048 ? 256 : 128;
     const size_t smem = (size_t)dv * sizeof(float);
     if (smem > 48 * 1024) return TNX_ERR_UNSUPPORTED;
-    const bool v8 = is_h16 && inv_freq_v && dv % 16 == 0 && D % 8 == 0 && out_ld % 8 == 0 && ((uintptr_t)att % 16) == 0 &&
+    const bool v8 = is_h16 && dv % (inv_freq_v ? 16 : 8) == 0 && (!gate || gate_per_head || (gate_ld % 8 == 0 && ((uintptr_t)gate % 16) == 0)) && D % 8 == 0 && out_ld % 8 == 0 && ((uintptr_t)att % 16) == 0 &&
                     ((uintptr_t)out % 16) == 0;
     if (is_h16 && v8)
         return tnx_launch_in_order(rotary_unrotate_kernel<h16, true>, dim3(n_tokens), dim3(threads), smem, stream, (const h16*)att,
-                                   token_request, positions, inv_freq_v, out_scale, (h16*)out, out_ld, H, dv, D);
+                                   token_request, positions, inv_freq_v, out_scale, (h16*)out, out_ld, H, dv, D, (const h16*)gate, gate_ld,
+                                   gate_per_head);
     if (is_h16)
         return tnx_launch_in_order(rotary_unrotate_kernel<h16, false>, dim3(n_tokens), dim3(threads), smem, stream, (const h16*)att,
-                                   token_request, positions, inv_freq_v, out_scale, (h16*)out, out_ld, H, dv, D);
+                                   token_request, positions, inv_freq_v, out_scale, (h16*)out, out_ld, H, dv, D, (const h16*)gate, gate_ld,
+                                   gate_per_head);
     return tnx_launch_in_order(rotary_unrotate_kernel<float, false>, dim3(n_tokens), dim3(threads), smem, stream, (const float*)att,
-                               token_request, positions, inv_freq_v, out_scale, (float*)out, out_ld, H, dv, D);
+                               token_request, positions, inv_freq_v, out_scale, (float*)out, out_ld, H, dv, D, (const float*)gate, gate_ld,
+                               gate_per_head);
 }

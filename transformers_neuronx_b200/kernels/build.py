@@ -55,6 +55,7 @@ SOURCES: Dict[str, str] = {
     "delta_rule": "delta_rule.cu",
     "ssd": "ssd.cu",
     "diff_attention": "diff_attention.cu",
+    "selective_scan": "selective_scan.cu",
 }
 
 _loaded: Dict[str, ctypes.CDLL] = {}

@@ -280,7 +280,19 @@ def mask_rule(window=0, chunk=0) -> int:
     return -chunk if chunk else window
 
 
-def attention_simt(q, cache, block_tables, token_request, positions, out, n_heads, scale, window=0, chunk=0):
+def _kept_and_bias(keep_first, bias, n_heads, window):
+    """The attention kernels' last arguments: how many first positions stay visible beside a window, and the distance
+    bias (mul, rate), 32-bit [n_heads] each: mul[h] * ln(1 + rate[h] * (i - j)) is taken off the scores (None: none)."""
+    keep_first = int(keep_first or 0)
+    if keep_first < 0 or (keep_first and not window):
+        raise KernelError("keep_first is a number of positions kept beside a window")
+    mul, rate = bias if bias is not None else (None, None)
+    _f32_vec(mul, "the bias's multiplier", n_heads); _f32_vec(rate, "the bias's rate", n_heads)
+    return c_int(keep_first), _p(mul), _p(rate)
+
+
+def attention_simt(q, cache, block_tables, token_request, positions, out, n_heads, scale, window=0, chunk=0, keep_first=0,
+                   bias=None):
     """q: [N, n_heads * head_dim] view; out likewise; cache as in kv_append."""
     lib = _lib("attention_simt", cache, q, out)
     _need(cache, "cache", _FLOATS, 5)
@@ -295,7 +307,8 @@ def attention_simt(q, cache, block_tables, token_request, positions, out, n_head
     _check(lib.tnx_attention_simt(_p(q), c_int(q_stride), _p(cache), _p(block_tables), c_int(block_tables.stride(0)),
                                   _p(token_request), _p(positions), _p(out), c_int(out_stride), c_int(N),
                                   c_int(n_heads), c_int(n_kv), c_int(d), c_int(ps), c_int(mask_rule(window, chunk)),
-                                  c_float(scale), c_int(_is_h16(cache)), _stream()), "attention_simt")
+                                  c_float(scale), *_kept_and_bias(keep_first, bias, n_heads, window),
+                                  c_int(_is_h16(cache)), _stream()), "attention_simt")
 
 
 def sample(logits, out, temperature=None, top_k=None, top_p=None, seeds=None, counters=None, suppress_id=-1,
@@ -624,7 +637,7 @@ def decode_attention_plan(pairs: int, sms: int, head_dim: int, max_pages: int):
 
 
 def attention_decode(q, cache, block_tables, token_request, positions, out, n_heads, scale, window=0, rows=None,
-                     n_rows=None, max_kv_len=None, n_splits=None, new_kv=None, warps=None, grouped=None, chunk=0):
+                     n_rows=None, max_kv_len=None, n_splits=None, new_kv=None, warps=None, grouped=None, chunk=0, keep_first=0, bias=None):
     """One query token per row over the paged 16-bit cache.  `rows` (int32) names the rows of q
     that are decode tokens (None: all); max_kv_len bounds their contexts (for the split plan).
     new_kv = (k, v), [rows of q, kv_heads * head_dim] bfloat16: the keys and values of the rows' own
@@ -647,6 +660,8 @@ def attention_decode(q, cache, block_tables, token_request, positions, out, n_he
     R = int(n_rows) if n_rows is not None else (rows.shape[0] if rows is not None else N)
     st = _state(q.device)
     max_pages = max(1, -(-(int(max_kv_len) if max_kv_len is not None else block_tables.shape[1] * ps) // ps))
+    if window or chunk:                                    # the kernel walks the pages that hold visible keys only
+        max_pages = min(max_pages, (int(window or chunk) - 1) // ps + 2 + -(-int(keep_first or 0) // ps))
     forced_warps, warps = warps, 4
     # with grouped key/value heads (2 or 4 query heads each) a block takes all query heads of a key/value head
     # Measured (32 query heads of 128 on 8 key/value heads, contexts of 2,048): the grouped form wins from 64 rows on
@@ -703,14 +718,14 @@ def attention_decode(q, cache, block_tables, token_request, positions, out, n_he
         _p(rows), _p(token_request), _p(positions), _p(out), c_int(out_stride), c_int(R),
         c_int(n_heads), c_int(n_kv), c_int(d), c_int(ps), c_int(mask_rule(window, chunk)), c_float(scale),
         c_int(n_splits), c_int(pps), _p(scratch), _p(st.get("att_counters")), _p(k_new), _p(v_new), c_int(kv_stride),
-        c_int(warps), c_int(heads_per_block), _stream()), "attention_decode")
+        c_int(warps), c_int(heads_per_block), *_kept_and_bias(keep_first, bias, n_heads, window), _stream()), "attention_decode")
 
 
 ATTN_PREFILL_TILE = 128      # query rows of one work item of the prefill attention kernel
 
 
 def attention_prefill(q, cache, block_tables, tile_req, tile_q0, q_start, q_len, ctx_len, out, n_heads, scale,
-                      window=0, n_items=None, chunk=0):
+                      window=0, n_items=None, chunk=0, keep_first=0, bias=None):
     """Causal attention of prompt portions: work items (request, first row of an ATTN_PREFILL_TILE-row tile)."""
     lib = _lib("attention_prefill", cache, q, out)
     _need(cache, "cache", _H16, 5)
@@ -726,7 +741,8 @@ def attention_prefill(q, cache, block_tables, tile_req, tile_q0, q_start, q_len,
     _check(lib.tnx_attention_prefill(_p(q), c_int(q_stride), _p(cache), _p(block_tables), c_int(block_tables.stride(0)),
                                      _p(tile_req), _p(tile_q0), _p(q_start), _p(q_len), _p(ctx_len), _p(out),
                                      c_int(out_stride), c_int(n), c_int(n_heads), c_int(n_kv), c_int(d), c_int(ps),
-                                     c_int(mask_rule(window, chunk)), c_float(scale), _stream()), "attention_prefill")
+                                     c_int(mask_rule(window, chunk)), c_float(scale),
+                                     *_kept_and_bias(keep_first, bias, n_heads, window), _stream()), "attention_prefill")
 
 
 def attention_prefill_tc_supported(q, cache, out) -> bool:
@@ -737,7 +753,7 @@ def attention_prefill_tc_supported(q, cache, out) -> bool:
 
 
 def attention_prefill_tc(q, cache, block_tables, tile_req, tile_q0, q_start, q_len, ctx_len, out, n_heads, scale,
-                         window=0, n_items=None, chunk=0):
+                         window=0, n_items=None, chunk=0, keep_first=0, bias=None):
     """attention_prefill on the tcgen05 tensor cores (head sizes 64 to 128 in steps of 16).  The cache must hold finite
     numbers in every row, written or not (CacheStorage allocates it zeroed)."""
     lib = _lib("attention_prefill_tc", cache, q, out)
@@ -756,10 +772,11 @@ def attention_prefill_tc(q, cache, block_tables, tile_req, tile_q0, q_start, q_l
                                         _p(block_tables), c_int(block_tables.stride(0)), _p(tile_req), _p(tile_q0),
                                         _p(q_start), _p(q_len), _p(ctx_len), _p(out), c_int(out_stride), c_int(n),
                                         c_int(n_heads), c_int(n_kv), c_int(d), c_int(ps), c_int(mask_rule(window, chunk)),
-                                        c_float(scale), _p(st["err"]), _stream()), "attention_prefill_tc")
+                                        c_float(scale), *_kept_and_bias(keep_first, bias, n_heads, window), _p(st["err"]),
+                                        _stream()), "attention_prefill_tc")
 
 
-def _attention_h16(ctx, group, q, cache, out, n_heads, scale, window, new_kv, chunk=0):
+def _attention_h16(ctx, group, q, cache, out, n_heads, scale, window, new_kv, chunk=0, keep_first=0, bias=None):
     if cache.shape[3] != 16 or cache.shape[4] > 256 or q.stride(0) % 8 or q.data_ptr() % 16:
         return False                             # rows wider than 256 dims: the CUDA-core kernel takes up to 768
     bt = ctx.block_tables[group]
@@ -774,32 +791,33 @@ def _attention_h16(ctx, group, q, cache, out, n_heads, scale, window, new_kv, ch
     if ctx.n_prefill_tiles:
         prefill = attention_prefill_tc if attention_prefill_tc_supported(q, cache, out) else attention_prefill
         prefill(q, cache, bt, ctx.tile_req, ctx.tile_q0, ctx.q_start, ctx.q_len, ctx.ctx_len, out,
-                n_heads, scale, window, n_items=ctx.n_prefill_tiles, chunk=chunk)
+                n_heads, scale, window, n_items=ctx.n_prefill_tiles, chunk=chunk, keep_first=keep_first, bias=bias)
     if ctx.n_decode_rows:
         attention_decode(q, cache, bt, ctx.token_request, ctx.positions, out, n_heads, scale, window,
                          rows=None if ctx.decode_only else ctx.decode_rows, n_rows=ctx.n_decode_rows,
-                         max_kv_len=ctx.max_decode_ctx, new_kv=fused, chunk=chunk)
+                         max_kv_len=ctx.max_decode_ctx, new_kv=fused, chunk=chunk, keep_first=keep_first, bias=bias)
     return True
 
 
 _attention_impls["h16"] = _attention_h16
 
 
-def attention(ctx, group, q, cache, out, n_heads, scale, window=0, new_kv=None, chunk=0):
+def attention(ctx, group, q, cache, out, n_heads, scale, window=0, new_kv=None, chunk=0, keep_first=0, bias=None):
     """Attention of this step's queries over the cache of the running schedule entry.  32-bit
     caches, and head sizes or windows that the 16-bit kernels do not take, run on the CUDA-core
     kernel; a 16-bit cache runs the prefill kernel for requests with several rows and the split
     decode kernel for requests with one.  new_kv = (k, v, slot_mapping): the keys and values of
     this step's tokens, not yet in the cache; they are appended here, by kv_append or (a step of
     decode tokens only, 16-bit) by the decode kernel itself; None: the cache holds them already (a mixer that
-    reads another mixer's pages).  window / chunk: see mask_rule."""
+    reads another mixer's pages).  window / chunk: see mask_rule; keep_first, bias: see
+    _kept_and_bias."""
     impl = _attention_impls.get("h16") if cache.dtype in _H16 else None
-    if impl is not None and impl(ctx, group, q, cache, out, n_heads, scale, window, new_kv, chunk):
+    if impl is not None and impl(ctx, group, q, cache, out, n_heads, scale, window, new_kv, chunk, keep_first, bias):
         return
     if new_kv is not None:
         kv_append(new_kv[0], new_kv[1], new_kv[2], cache, ctx.page_size)
     attention_simt(q, cache, ctx.block_tables[group], ctx.token_request, ctx.positions, out, n_heads, scale,
-                   window, chunk)
+                   window, chunk, keep_first, bias)
 
 
 # ---------------------------------------------------------------------------------------------
@@ -956,9 +974,9 @@ def conv_qkv_prep(proj, col0, conv_w, taps, state, ctx, q_norm, k_norm, eps, inv
 
 
 def moe_route(h, router, token_request, ids, weights, top, softmax_scores=False, renormalize=False, correction=None,
-              n_groups=1, keep_groups=1, group_top=2, renorm_eps=0.0, weight_scale=1.0):
+              n_groups=1, keep_groups=1, group_top=2, renorm_eps=0.0, weight_scale=1.0, bias=None):
     """For every row of h [N, W]: the `top` experts with the largest scores (sigmoid, or softmax, of the 32-bit product
-    with router [E, W]) into ids [N, top] (int32; -1 for a padded row) and their scores into weights [N, top].
+    with router [E, W], plus bias [E] where it is given) into ids [N, top] (int32; -1 for a padded row) and their scores into weights [N, top].
     correction (32-bit [E]): added to the sigmoid scores for the choice only.  n_groups > 1: the experts form equal groups
     of neighbours, a group's score is the sum of its group_top largest choice scores, and only experts of the keep_groups
     best groups can be chosen.  The weights are divided by (their sum + renorm_eps) with `renormalize`, then multiplied
@@ -974,11 +992,11 @@ def moe_route(h, router, token_request, ids, weights, top, softmax_scores=False,
     _need(ids, "ids", torch.int32, 2); _need(weights, "weights", torch.float32, 2)
     if tuple(ids.shape) != (N, top) or tuple(weights.shape) != (N, top):
         raise KernelError(f"ids and weights must be [{N}, {top}]")
-    _f32_vec(correction, "correction", E)
+    _f32_vec(correction, "correction", E); _f32_vec(bias, "bias", E)
     _check(lib.tnx_moe_route(_p(h), c_int(ld), _p(router), _p(token_request), _p(ids), _p(weights), c_int(N), c_int(W),
                              c_int(E), c_int(top), c_int(1 if softmax_scores else 0), c_int(1 if renormalize else 0),
                              c_int(_is_h16(h)), c_int(_is_h16(router)), _p(correction), c_int(n_groups), c_int(keep_groups),
-                             c_int(group_top), c_float(renorm_eps), c_float(weight_scale), _stream()), "moe_route")
+                             c_int(group_top), c_float(renorm_eps), c_float(weight_scale), _p(bias), _stream()), "moe_route")
 
 
 EXPERT_FORMS = {"gated_swish": 0, "relu2": 1}
@@ -1136,11 +1154,13 @@ def moe_combine(lib, per_pair, row_of_pair, weights, out, accumulate, weight_on_
 
 
 def rotary_qkv_prep(proj, q_off, k_off, v_off, token_request, positions, q_weight, k_weight, eps, head_scale,
-                    inv_freq_qk, rot_dims, inv_freq_v, q_out, k_out, v_out, n_heads, n_kv_heads, k_dim, v_dim, pad_dim):
+                    inv_freq_qk, rot_dims, inv_freq_v, q_out, k_out, v_out, n_heads, n_kv_heads, k_dim, v_dim, pad_dim,
+                    other_values=None, mix_weight=None):
     """From one product's output `proj` [N, *] (queries at column q_off, keys at k_off, values at v_off): the
     queries and keys normalised over the whole projection (where a weight is given), rotated by position
     on their first rot_dims dims, the queries multiplied by their head's number; the values rotated over
-    all their dims (where inv_freq_v is given); each written with pad_dim dims a head, the rest zero."""
+    all their dims (where inv_freq_v is given); each written with pad_dim dims a head, the rest zero.
+    other_values [N, n_kv_heads * v_dim] with mix_weight (32-bit [1]): the values become (1 - w) v + w other."""
     lib = _lib("rotary_qkv", proj, q_out)
     _need(proj, "proj", _FLOATS, None, contiguous=False)
     N, width, ld = _rows_2d(proj, "proj")
@@ -1155,17 +1175,25 @@ def rotary_qkv_prep(proj, q_off, k_off, v_off, token_request, positions, q_weigh
     _f32_vec(inv_freq_qk, "inv_freq_qk", rot_dims // 2 if rot_dims else None); _f32_vec(inv_freq_v, "inv_freq_v", dv // 2)
     _need(token_request, "token_request", torch.int32, 1)
     _need(positions, "positions", torch.int32, 1)
+    other_ld = 0
+    if other_values is not None:
+        _need(other_values, "other_values", proj.dtype, None, contiguous=False)
+        No, wo, other_ld = _rows_2d(other_values, "other_values")
+        if (No, wo) != (N, G * dv) or inv_freq_v is not None:
+            raise KernelError(f"other_values must be [{N}, {G * dv}] and the values not rotated")
+        _need(mix_weight, "mix_weight", torch.float32, 1)
     _check(lib.tnx_rotary_qkv_prep(_p(proj), c_int(ld), c_int(q_off), c_int(k_off), c_int(v_off), _p(token_request),
                                    _p(positions), _p(q_weight), _p(k_weight), c_float(eps), _p(head_scale),
                                    _p(inv_freq_qk), c_int(rot_dims), _p(inv_freq_v), _p(q_out), _p(k_out), _p(v_out),
-                                   c_int(N), c_int(H), c_int(G), c_int(dk), c_int(dv), c_int(D), c_int(_is_h16(proj)),
-                                   _stream()), "rotary_qkv_prep")
+                                   c_int(N), c_int(H), c_int(G), c_int(dk), c_int(dv), c_int(D), _p(other_values),
+                                   c_int(other_ld), _p(mix_weight), c_int(_is_h16(proj)), _stream()), "rotary_qkv_prep")
 
 
-def rotary_unrotate(att, token_request, positions, inv_freq_v, out_scale, out, n_heads, v_dim, pad_dim):
+def rotary_unrotate(att, token_request, positions, inv_freq_v, out_scale, out, n_heads, v_dim, pad_dim, gate=None):
     """att [N, n_heads * pad_dim]: each head's first v_dim dims turned back by the token's position (pair m with
     m + v_dim/2, by -p * inv_freq_v[m]; no turn without inv_freq_v), times out_scale, written v_dim a head into
-    `out` [N, n_heads * v_dim] (a column slice of a wider buffer is allowed)."""
+    `out` [N, n_heads * v_dim] (a column slice of a wider buffer is allowed).  gate: a view [N, n_heads] or
+    [N, n_heads * v_dim] in att's type whose sigmoid multiplies each head's dims, or each dim."""
     lib = _lib("rotary_qkv", att, out)
     _need(att, "att", _FLOATS, 2)
     N = att.shape[0]
@@ -1176,14 +1204,23 @@ def rotary_unrotate(att, token_request, positions, inv_freq_v, out_scale, out, n
     if (No, wo) != (N, n_heads * v_dim):
         raise KernelError(f"out must be [{N}, {n_heads * v_dim}]")
     _f32_vec(inv_freq_v, "inv_freq_v", v_dim // 2)
+    gate_ld = per_head = 0
+    if gate is not None:
+        _need(gate, "gate", att.dtype, None, contiguous=False)
+        Ng, wg, gate_ld = _rows_2d(gate, "gate")
+        if Ng != N or wg not in (n_heads, n_heads * v_dim) or inv_freq_v is not None:
+            raise KernelError(f"a gate must be [{N}, {n_heads}] or [{N}, {n_heads * v_dim}] and the values not rotated")
+        per_head = 1 if wg == n_heads else 0
     _check(lib.tnx_rotary_unrotate(_p(att), _p(token_request), _p(positions), _p(inv_freq_v), c_float(out_scale),
-                                   _p(out), c_int(out_ld), c_int(N), c_int(n_heads), c_int(v_dim), c_int(pad_dim),
-                                   c_int(_is_h16(att)), _stream()), "rotary_unrotate")
+                                   _p(out), c_int(out_ld), c_int(N), c_int(n_heads), c_int(v_dim), c_int(pad_dim), _p(gate),
+                                   c_int(gate_ld), c_int(per_head), c_int(_is_h16(att)), _stream()), "rotary_unrotate")
 
 
-def retention_prep(proj, q_off, k_off, token_request, positions, inv_freq, rot_dims, k_scale, q_out, k_out, n_heads, k_dim):
+def retention_prep(proj, q_off, k_off, token_request, positions, inv_freq, rot_dims, k_scale, q_out, k_out, n_heads, k_dim,
+                   activation=None, v_off=0, v_out=None):
     """32-bit queries and keys [N, n_heads * k_dim] for the retention scan: rotated by position on their first
-    rot_dims dims, the keys then multiplied by k_scale."""
+    rot_dims dims, the keys then multiplied by k_scale.  `activation` is applied to queries and keys first, and to the values
+    at column v_off, which v_out [N, *] (32-bit) then receives."""
     lib = _lib("retention", proj)
     _need(proj, "proj", _FLOATS, None, contiguous=False)
     N, width, ld = _rows_2d(proj, "proj")
@@ -1194,9 +1231,16 @@ def retention_prep(proj, q_off, k_off, token_request, positions, inv_freq, rot_d
         if tuple(t.shape) != (N, n_heads * k_dim):
             raise KernelError(f"{nm} must be [{N}, {n_heads * k_dim}]")
     _f32_vec(inv_freq, "inv_freq", rot_dims // 2 if rot_dims else None)
+    n_values = 0
+    if v_out is not None:
+        _need(v_out, "v_out", torch.float32, 2)
+        n_values = v_out.shape[1]
+        if v_out.shape[0] != N or v_off + n_values > width:
+            raise KernelError("v_out does not fit the projection's value columns")
     _check(lib.tnx_retention_prep(_p(proj), c_int(ld), c_int(q_off), c_int(k_off), _p(token_request), _p(positions),
                                   _p(inv_freq), c_int(rot_dims), c_float(k_scale), _p(q_out), _p(k_out), c_int(N),
-                                  c_int(n_heads), c_int(k_dim), c_int(_is_h16(proj)), _stream()), "retention_prep")
+                                  c_int(n_heads), c_int(k_dim), c_int(activation_code(activation)), c_int(v_off), _p(v_out),
+                                  c_int(n_values), c_int(_is_h16(proj)), _stream()), "retention_prep")
 
 
 def retention_scan(q, k, v, decay, state, q_start, q_len, state_slots, out, n_heads, k_dim, v_dim, most_tokens=None,
@@ -1247,12 +1291,14 @@ def retention_scan(q, k, v, decay, state, q_start, q_len, state_slots, out, n_he
 
 
 def retention_decode(proj, q_off, k_off, v_off, g_off, positions, inv_freq, rot_dims, k_scale, decay, state, q_start, q_len,
-                     state_slots, eps, out_scale, out, n_heads, k_dim, v_dim) -> bool:
+                     state_slots, eps, out_scale, out, n_heads, k_dim, v_dim, activation=None, gate_activation="silu",
+                     raw=False) -> bool:
     """A step in which every request has ONE row: retention_prep, retention_scan and headwise_gated_rms_norm in one
     kernel (the 32-bit queries, keys and outputs never pass through memory).  Returns False, having launched nothing,
     for sizes the kernel does not take (k_dim or v_dim no multiple of four, very wide heads): the caller then runs the
-    three kernels.  g_off None: no gate."""
-    lib = _lib("retention", proj, out)
+    three kernels.  g_off None: no gate.  `activation`: of queries, keys and values.  raw: `out` is 32-bit and receives
+    the recurrence's output as it is (no norm, gate or scale)."""
+    lib = _lib("retention", proj)
     _need(proj, "proj", _FLOATS, None, contiguous=False)
     N, width, ld = _rows_2d(proj, "proj")
     offs = [q_off + n_heads * k_dim, k_off + n_heads * k_dim, v_off + n_heads * v_dim] + \
@@ -1262,7 +1308,7 @@ def retention_decode(proj, q_off, k_off, v_off, g_off, positions, inv_freq, rot_
     _need(state, "state", torch.float32, 4)
     if tuple(state.shape[1:]) != (n_heads, v_dim, k_dim):
         raise KernelError(f"state must be [slots, {n_heads}, {v_dim}, {k_dim}]")
-    _need(out, "out", proj.dtype, None, contiguous=False)
+    _need(out, "out", torch.float32 if raw else proj.dtype, None, contiguous=False)
     No, wo, out_ld = _rows_2d(out, "out")
     if (No, wo) != (N, n_heads * v_dim):
         raise KernelError(f"out must be [{N}, {n_heads * v_dim}]")
@@ -1274,7 +1320,8 @@ def retention_decode(proj, q_off, k_off, v_off, g_off, positions, inv_freq, rot_
                                     c_int(-1 if g_off is None else g_off), _p(positions), _p(inv_freq), c_int(rot_dims),
                                     c_float(k_scale), _p(decay), _p(state), _p(q_start), _p(q_len), _p(state_slots),
                                     c_float(eps), c_float(out_scale), _p(out), c_int(out_ld), c_int(q_len.shape[0]),
-                                    c_int(n_heads), c_int(k_dim), c_int(v_dim), c_int(_is_h16(proj)), _stream())
+                                    c_int(n_heads), c_int(k_dim), c_int(v_dim), c_int(activation_code(activation)),
+                                    c_int(activation_code(gate_activation)), c_int(1 if raw else 0), c_int(_is_h16(proj)), _stream())
     if code == -2:
         return False
     _check(code, "retention_decode")
@@ -1288,6 +1335,29 @@ def retention_scan_force(lanes=0, stage_tokens=0, dtype=None) -> None:
     lib = _build.load("retention", dtype if dtype in _H16 else None)
     if lib.tnx_retention_scan_force(c_int(int(lanes)), c_int(int(stage_tokens))) != 0:
         raise KernelError(f"retention_scan_force: {lanes} lanes (0 or 16) and stages of {stage_tokens} tokens (0 to 32) are not a choice")
+
+
+def gated_rms_norm(o, gate, token_request, weight, eps, out_scale, out, gate_activation="sigmoid"):
+    """out = o / rms(o over the whole row) (* weight) * act(gate) * out_scale; o 32-bit [N, width], gate (optional) and out
+    views in the activation type."""
+    lib = _lib("retention", gate, out)
+    _need(o, "o", torch.float32, 2)
+    N, width = o.shape
+    gate_ld = 0
+    if gate is not None:
+        _need(gate, "gate", out.dtype, None, contiguous=False)
+        Ng, wg, gate_ld = _rows_2d(gate, "gate")
+        if (Ng, wg) != (N, width):
+            raise KernelError(f"gate must be [{N}, {width}]")
+    _need(out, "out", _FLOATS, None, contiguous=False)
+    No, wo, out_ld = _rows_2d(out, "out")
+    if (No, wo) != (N, width):
+        raise KernelError(f"out must be [{N}, {width}]")
+    _f32_vec(weight, "weight", width)
+    _need(token_request, "token_request", torch.int32, 1)
+    _check(lib.tnx_gated_rms_norm(_p(o), _p(gate), c_int(gate_ld), _p(token_request), _p(weight), c_float(eps),
+                                  c_float(out_scale), _p(out), c_int(out_ld), c_int(N), c_int(width),
+                                  c_int(activation_code(gate_activation)), c_int(_is_h16(out)), _stream()), "gated_rms_norm")
 
 
 def headwise_gated_rms_norm(o, gate, token_request, weight, eps, out_scale, out, n_heads, v_dim, gate_activation="silu"):
@@ -1374,6 +1444,66 @@ def ssd_gate_norm(y, x, skip, z, token_request, weight, eps, activation, out, v_
     _check(lib.tnx_ssd_gate_norm(_p(y), _p(x), _p(skip), _p(z), c_int(z_ld), _p(token_request), _p(weight), c_float(eps),
                                  c_int(activation_code(activation)), _p(out), c_int(out_ld), c_int(N), c_int(inner),
                                  c_int(v_dim), c_int(parts), c_int(_is_h16(out)), _stream()), "ssd_gate_norm")
+
+
+def causal_conv(proj, col0, conv_w, conv_b, taps, state, ctx, activation, out):
+    """out [N, channels] (in proj's type): the columns col0 .. of `proj` through a short causal convolution per channel
+    (conv_w [taps, channels], conv_b [channels] or None, both 32-bit) and the activation; the past comes from this step's
+    rows or from `state` [slots, taps - 1, channels] in proj's type, which is brought up to date."""
+    lib = _lib("selective_scan", proj, out)
+    _need(proj, "proj", _FLOATS, None, contiguous=False)
+    N, width, ld = _rows_2d(proj, "proj")
+    _need(out, "out", proj.dtype, 2)
+    C = out.shape[1]
+    if out.shape[0] != N or col0 < 0 or col0 + C > width:
+        raise KernelError("the projection is narrower than its convolved columns")
+    _need(conv_w, "conv_w", torch.float32, 2)
+    if tuple(conv_w.shape) != (taps, C):
+        raise KernelError(f"conv_w must be [{taps}, {C}]")
+    _f32_vec(conv_b, "conv_b", C)
+    if taps > 1:
+        _need(state, "state", proj.dtype, 3)
+        if tuple(state.shape[1:]) != (taps - 1, C):
+            raise KernelError(f"state must be [slots, {taps - 1}, {C}]")
+    for t, nm in ((ctx.token_request, "token_request"), (ctx.positions, "positions"), (ctx.q_start, "q_start"),
+                  (ctx.q_len, "q_len"), (ctx.state_slots, "state_slots")):
+        _need(t, nm, torch.int32, 1)
+    _check(lib.tnx_causal_conv(_p(proj), c_int(ld), c_int(col0), _p(conv_w), _p(conv_b), c_int(taps),
+                               _p(state if taps > 1 else None), _p(ctx.token_request), _p(ctx.positions), _p(ctx.q_start),
+                               _p(ctx.q_len), _p(ctx.state_slots), c_int(activation_code(activation)), _p(out), c_int(N),
+                               c_int(C), c_int(_is_h16(proj)), _stream()), "causal_conv")
+    if taps > 1 and not ctx.decode_only:
+        conv_state_update(proj, col0, state, ctx)
+
+
+def selective_scan(x, dt, low, b_off, c_off, decay_log2, dt_bias, skip, z, state, ctx, activation, out):
+    """Per channel c and state n, token by token for every request of the step: dt <- softplus(dt + dt_bias),
+    S[c, n] <- 2^(decay_log2[c, n] dt_c) S[c, n] + dt_c x_c B_n, out_c = (sum_n S[c, n] C_n + skip_c x_c) * act(z_c).
+    x, z, out: views [N, C] in the activation type; dt 32-bit [N, C]; B and C the state-many columns of `low` at b_off and
+    c_off; state 32-bit [slots, C, n], decay_log2 32-bit [C, n]."""
+    lib = _lib("selective_scan", x, out)
+    _need(state, "state", torch.float32, 3)
+    _, C, Ns = state.shape
+    _need(dt, "dt", torch.float32, 2)
+    N = dt.shape[0]
+    lds = []
+    for t, nm, w in ((x, "x", C), (z, "z", C), (out, "out", C), (low, "low", None)):
+        _need(t, nm, x.dtype, None, contiguous=False)
+        n, wd, ld = _rows_2d(t, nm)
+        if n != N or (w is not None and wd != w):
+            raise KernelError(f"{nm} must be [{N}, {w}]")
+        lds.append(ld)
+    if dt.shape[1] != C or tuple(decay_log2.shape) != (C, Ns) or max(b_off, c_off) + Ns > low.shape[1] or min(b_off, c_off) < 0:
+        raise KernelError("dt, decay_log2 or low do not fit the state's channels")
+    _need(decay_log2, "decay_log2", torch.float32, 2)
+    _f32_vec(dt_bias, "dt_bias", C); _f32_vec(skip, "skip", C)
+    for t, nm in ((ctx.q_start, "q_start"), (ctx.q_len, "q_len"), (ctx.state_slots, "state_slots")):
+        _need(t, nm, torch.int32, 1)
+    _check(lib.tnx_selective_scan(_p(x), c_int(lds[0]), _p(dt), _p(low), c_int(lds[3]), c_int(b_off), c_int(c_off),
+                                  _p(decay_log2), _p(dt_bias), _p(skip), _p(z), c_int(lds[1]), _p(state), _p(ctx.q_start),
+                                  _p(ctx.q_len), _p(ctx.state_slots), c_int(activation_code(activation)), _p(out),
+                                  c_int(lds[2]), c_int(ctx.q_len.shape[0]), c_int(C), c_int(Ns),
+                                  c_int(1 if ctx.decode_only else N), c_int(_is_h16(x)), _stream()), "selective_scan")
 
 
 def diff_qkv_prep(proj, col0, token_request, positions, q_norm, k_norm, eps, temp_coef, temp_every, q_out, k_out, v_out,

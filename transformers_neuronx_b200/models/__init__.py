@@ -4,3 +4,4 @@ from . import vononex  # noqa: F401  registers Vononex
 from . import pifelix  # noqa: F401  registers Pifelix
 from . import tutelix  # noqa: F401  registers Tutelix
 from . import vozirax  # noqa: F401  registers Vozirax
+from . import resatar  # noqa: F401  registers Resatar

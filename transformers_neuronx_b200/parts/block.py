@@ -17,7 +17,8 @@ output_norm:                                              x = x + m norm1(mixer(
 sandwich_norm:                                            x = x + norm1_post(mixer(norm1(x))); x = x + norm2_post(ff(norm2(x)))
     a norm before and after each sublayer (the layer's spec names the two further norms).  The sublayer's result
     goes into a 32-bit buffer; one kernel normalises it, adds it to the stream and, where the next sublayer of the
-    same layer follows, applies that sublayer's input norm to the new row (Norm.forward_add(..., then=norm2)).
+    same layer follows, applies that sublayer's input norm to the new row (Norm.forward_add(..., then=norm2)).  Where
+    a layer of the same kind follows, the kernel that closes this one forms that layer's first input the same way.
 
 parallel_residual:                                        x = x + s1 * mixer(norm1(x)) + s2 * ff(norm2(x))
     both sublayers read the same x, each behind a norm of its own (one kernel forms both norms: the mean square of a row
@@ -161,17 +162,31 @@ class SandwichNormBlock(ScaledPostNormBlock):
 
     def forward(self, ctx, x, x_act):
         N, W = x.shape
-        h = ctx.scratch(N, W)
-        self.norm1.forward(ctx, x, out_act=h)
+        handed, ctx.handed_on = getattr(ctx, "handed_on", None), None
+        h1 = None
+        if handed is not None and handed[0] == ctx.entry_index and handed[1] is self:
+            h1 = handed[2]                         # the block before formed it in the kernel that closed its layer
+        if h1 is None:
+            h1 = ctx.scratch(N, W)
+            self.norm1.forward(ctx, x, out_act=h1)
         out = ctx.scratch(N, W, x.dtype)
-        self._run(ctx, self.mixer, h, out)
+        self._run(ctx, self.mixer, h1, out)
         if self.feed_forward is None:
-            self.norm1_post.forward_add(ctx, x, 1.0, out, out_f32=x)
+            self._close(ctx, x, out, self.norm1_post)
             return
+        h = ctx.scratch(N, W)
         # one kernel: the stream takes the normalised mixer output, and the new row is normalised for the feed-forward
         self.norm1_post.forward_add(ctx, x, 1.0, out, out_f32=x, out_act=h, then=self.norm2)
         self._run(ctx, self.feed_forward, h, out)
-        self.norm2_post.forward_add(ctx, x, 1.0, out, out_f32=x)
+        self._close(ctx, x, out, self.norm2_post)
+
+    def _close(self, ctx, x, out, norm):
+        """The layer's last sum; the layer that follows, if it is of this kind, gets its first norm from the same kernel."""
+        nxt, h = getattr(ctx, "next_block", None), None
+        if isinstance(nxt, SandwichNormBlock) and type(nxt.norm1) is type(norm):
+            h = ctx.carry(("sandwich", (ctx.entry_index + 1) & 1), x.shape[0], x.shape[1])
+            ctx.handed_on = (ctx.entry_index + 1, nxt, h)
+        norm.forward_add(ctx, x, 1.0, out, out_f32=x, out_act=h, then=nxt.norm1 if h is not None else None)
 
 
 class ChannelScale(Part):

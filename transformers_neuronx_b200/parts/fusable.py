@@ -36,6 +36,11 @@ def fuse_linears_along_k(parts: List[Linear], scales, device) -> Linear:
     return fused
 
 
+def pitched(ctx, rows, cols):
+    """A scratch buffer [rows, cols] whose row pitch is a multiple of 8 elements."""
+    return ctx.scratch(rows, -(-cols // 8) * 8)[:, :cols]
+
+
 class FusableMixer(Mixer):
     """Subclasses set self.inputs (list of Linear reading h), self.output (Linear) and implement
     inner_width, load_extras(), mix()."""
@@ -96,9 +101,14 @@ class FusableMixer(Mixer):
     def parameter_bytes(self):
         return self._fused_in.parameter_bytes() + self.output.parameter_bytes() + self.extra_parameter_bytes()
 
+    def projection_buffer(self, ctx, rows):
+        """Where this mixer's projections go when it runs alone: rows of a multiple of 8 columns, so that a few columns at
+        the end (a gate's) leave every row on a 16-byte boundary."""
+        return pitched(ctx, rows, self.projection_width)
+
     def forward(self, ctx, h, out, accumulate=True):
         N = h.shape[0]
-        proj = ctx.scratch(N, self.projection_width)
+        proj = self.projection_buffer(ctx, N)
         self._fused_in.forward(h, proj)
         inner = ctx.scratch(N, self.inner_width)
         self.mix(ctx, proj, 0, inner, 1.0)

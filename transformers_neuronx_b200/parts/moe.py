@@ -1,5 +1,5 @@
 """A feed-forward of routed experts: each token runs `top` of `n_experts` small feed-forwards (gated, or
-down(relu(up x)^2) without a gate; the router may add a correction to the scores for the choice only, restrict the choice
+down(relu(up x)^2) without a gate; the router may have a bias, add a correction to the scores for the choice only, restrict the choice
 to the best groups of experts, and scale the weights: parts/spec.py: RoutedFeedForwardSpec).
 
   z = W_router h (32-bit sums), s = sigmoid(z) or softmax(z); the `top` largest scores choose the experts
@@ -7,6 +7,7 @@ to the best groups of experts, and scale the weights: parts/spec.py: RoutedFeedF
   expert(x) = W_down (g * sigmoid(act_alpha g) * (u + up_shift)),  g = min(W_gate x, gate_limit),
               u = clamp(W_up x, -up_limit, up_limit)
   result = sum_j expert_{e_j}(w_j h)  (weight_on_input)   or   sum_j w_j expert_{e_j}(h)
+           (+ shared(h), a gated feed-forward that every token runs)
 
 The experts' matrices are kept stacked, [E, 2 ff, hidden] (gate rows, then up rows) and [E, hidden, ff], in the type
 they are stored in.  A step routes on the device (no read on the host: the part is graph-safe) and then takes one of
@@ -23,14 +24,18 @@ import torch
 from ..kernels import ops
 from ..weights.loader import TensorSpec
 from .base import FeedForward, to_device, weight_to_device
-from .registry import register_feed_forward
+from .registry import build_part, register_feed_forward
 from .spec import RoutedFeedForwardSpec
 
 
 class RoutedExperts(FeedForward):
     graph_safe = True
     can_overwrite = True
-    libraries = ("moe", "moe_grouped", "gemm_tc")
+
+    @property
+    def libraries(self):
+        return ("moe", "moe_grouped", "gemm_tc") + (tuple(self.shared.libraries) if self.shared is not None else ())
+
     # Rows from which the grouped tensor-core form runs in a 16-bit engine.  Measured at width 2048 (8 experts of inner
     # width 2816, 2 a token): a decode step of 1 / 8 / 32 requests takes 0.48 / 0.75 / 1.03 ms with it and 0.52 / 1.10 /
     # 2.54 ms with the kernels that stream the matrices through the multiply-add units, so it always runs.
@@ -55,24 +60,31 @@ class RoutedExperts(FeedForward):
             raise ValueError(f"the {s.keep_groups} kept groups hold fewer than {s.top} experts")
         if (s.correction or s.n_groups > 1) and s.scores != "sigmoid":
             raise ValueError("a correction of the choice and groups of experts go with sigmoid scores")
-        self.router = self.gate_up = self.down = self.correction = None
+        self.shared = build_part("feed_forward", s.shared)
+        self.router = self.gate_up = self.down = self.correction = self.router_bias = None
 
     def tensor_specs(self):
         s = self.spec
         out = [TensorSpec(s.router, (s.n_experts, s.hidden), "matrix")]
         if s.correction:
             out.append(TensorSpec(s.correction, (s.n_experts,), "bias"))
+        if s.router_bias:
+            out.append(TensorSpec(s.router_bias, (s.n_experts,), "bias"))
         for e in s.experts:
             if self.gated:
                 out.append(TensorSpec(e.gate, (s.ff, s.hidden), "matrix"))
             out += [TensorSpec(e.up, (s.ff, s.hidden), "matrix"), TensorSpec(e.down, (s.hidden, s.ff), "matrix")]
-        return out
+        return out + (self.shared.tensor_specs() if self.shared is not None else [])
 
     def load(self, tensors, device, act_dtype):
         s = self.spec
         self.router = weight_to_device(tensors[s.router], device, act_dtype, s.router)
         if s.correction:
             self.correction = to_device(tensors[s.correction], device, torch.float32)
+        if s.router_bias:
+            self.router_bias = to_device(tensors[s.router_bias], device, torch.float32)
+        if self.shared is not None:
+            self.shared.load(tensors, device, act_dtype)
         first = weight_to_device(tensors[s.experts[0].up], device, act_dtype, s.experts[0].up)
         # gate rows, then up rows; experts without a gate: the up rows alone
         self.gate_up = torch.empty((s.n_experts, (2 if self.gated else 1) * s.ff, s.hidden), dtype=first.dtype, device=device)
@@ -87,8 +99,8 @@ class RoutedExperts(FeedForward):
                 dst.copy_(w)
 
     def parameter_bytes(self):
-        return sum(t.numel() * t.element_size() for t in (self.router, self.gate_up, self.down, self.correction)
-                   if t is not None)
+        return sum(t.numel() * t.element_size() for t in (self.router, self.gate_up, self.down, self.correction, self.router_bias)
+                   if t is not None) + (self.shared.parameter_bytes() if self.shared is not None else 0)
 
     def step_bytes(self, n_tokens: int) -> int:
         """Bytes of weights a step of n_tokens is expected to read: every expert once that some token chooses, with
@@ -96,7 +108,8 @@ class RoutedExperts(FeedForward):
         s = self.spec
         used = s.n_experts * (1.0 - (1.0 - s.top / s.n_experts) ** n_tokens)
         per = (self.gate_up[0].numel() + self.down[0].numel()) * self.gate_up.element_size()
-        return int(self.router.numel() * self.router.element_size() + used * per)
+        return int(self.router.numel() * self.router.element_size() + used * per) + \
+            (self.shared.parameter_bytes() if self.shared is not None else 0)
 
     def forward(self, ctx, h, out, accumulate=True):
         s, N = self.spec, h.shape[0]
@@ -104,18 +117,20 @@ class RoutedExperts(FeedForward):
         weights = ctx.scratch(N, s.top, torch.float32)
         ops.moe_route(h, self.router, ctx.token_request, ids, weights, s.top, softmax_scores=s.scores == "softmax",
                       renormalize=s.renormalize, correction=self.correction, n_groups=s.n_groups, keep_groups=s.keep_groups,
-                      group_top=s.group_top, renorm_eps=s.renorm_eps, weight_scale=s.weight_scale)
+                      group_top=s.group_top, renorm_eps=s.renorm_eps, weight_scale=s.weight_scale, bias=self.router_bias)
         inf = math.inf
         limits = (s.gate_limit if s.gate_limit is not None else inf, -s.up_limit if s.up_limit is not None else -inf,
                   s.up_limit if s.up_limit is not None else inf)
         if N >= self.GROUPED_FROM and ops.moe_grouped_supported(h, self.gate_up, self.down):
             ops.moe_grouped(ctx, h, self.gate_up, self.down, ids, weights, out, *limits, s.act_alpha, s.up_shift,
                             weight_on_input=s.weight_on_input, accumulate=accumulate, form=s.expert_form)
-            return
-        y = ctx.scratch(N * s.top, s.ff)
-        ops.moe_experts(h, self.gate_up, self.down, ids, weights, y, out, *limits, s.act_alpha, s.up_shift,
-                        weight_on_input=s.weight_on_input, accumulate=accumulate,
-                        per_pair=ctx.scratch(N * s.top, s.hidden, torch.float32), form=s.expert_form)
+        else:
+            y = ctx.scratch(N * s.top, s.ff)
+            ops.moe_experts(h, self.gate_up, self.down, ids, weights, y, out, *limits, s.act_alpha, s.up_shift,
+                            weight_on_input=s.weight_on_input, accumulate=accumulate,
+                            per_pair=ctx.scratch(N * s.top, s.hidden, torch.float32), form=s.expert_form)
+        if self.shared is not None:
+            self.shared.forward(ctx, h, out)
 
 
 register_feed_forward("routed_experts", RoutedExperts)

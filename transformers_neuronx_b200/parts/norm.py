@@ -1,6 +1,7 @@
 """Norms over the hidden axis.
 
-RMS norm: y / sqrt(mean(y^2) + eps) * (weight + weight_offset), in 32-bit; it can normalise a sum
+RMS norm: y / sqrt(mean(y^2) + eps) * (weight + weight_offset), in 32-bit, the weight a vector over the hidden axis or
+one number for all of it; it can normalise a sum
 y = x_scale * x + delta in the same kernel, which is what a post-norm block with a scaled residual asks for,
 or normalise a sublayer's output alone and add it to the stream (x + add_scale * norm(delta)).
 
@@ -62,11 +63,13 @@ class RMSNorm(Norm):
 
     def tensor_specs(self):
         s = self.spec
-        return [TensorSpec(s.weight, (s.size,), "norm_weight")] if s.weight else []
+        return [TensorSpec(s.weight, () if s.one_number else (s.size,), "norm_weight")] if s.weight else []
 
     def load(self, tensors, device, act_dtype):
         s = self.spec
         self.weight = to_device(tensors[s.weight], device, torch.float32) if s.weight else None
+        if s.weight and s.one_number:                 # the kernels take a vector
+            self.weight = self.weight.reshape(1).expand(s.size).contiguous()
 
     def parameter_bytes(self):
         return self.weight.numel() * 4 if self.weight is not None else 0

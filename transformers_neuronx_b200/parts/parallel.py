@@ -8,7 +8,7 @@ keeps its own cache: the part's cache_need() is the tuple of the branches' needs
 """
 from __future__ import annotations
 
-from .fusable import FusableMixer, fuse_linears_along_k
+from .fusable import FusableMixer, fuse_linears_along_k, pitched
 from .linear import fuse_linears
 from .registry import build_part, register_mixer
 from .spec import ParallelMixerSpec
@@ -57,9 +57,9 @@ class ParallelMixer(FusableMixer):
 
     def forward(self, ctx, h, out, accumulate=True):
         N = h.shape[0]
-        proj = ctx.scratch(N, self._fused_in.spec.out_features)
+        proj = pitched(ctx, N, self._fused_in.spec.out_features)
         self._fused_in.forward(h, proj)
-        inner = ctx.scratch(N, self._fused_out.spec.in_features)
+        inner = pitched(ctx, N, self._fused_out.spec.in_features)
         col = k0 = 0
         for j, (b, s) in enumerate(zip(self.branches, self.scales)):
             b.mix(ctx, proj, col, inner[:, k0:k0 + b.inner_width], s, sub=j)

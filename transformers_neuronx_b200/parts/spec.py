@@ -28,6 +28,7 @@ class NormSpec:
     weight: Optional[str] = None     # None: no elementwise scale
     bias: Optional[str] = None
     weight_offset: float = 0.0       # 'rms_norm': the scale is weight + weight_offset (1.0: "one plus" weights)
+    one_number: bool = False         # 'rms_norm': the stored weight is a single number (shape []) for all coordinates
 
 
 @dataclass(frozen=True)
@@ -43,13 +44,24 @@ class FrequencyRampSpec:
 
 
 @dataclass(frozen=True)
+class FrequencyBandsSpec:
+    """Stretching of a rotation's frequencies by wave length l = 2 pi / f: f stays where l < original / high, becomes
+    f / factor where l > original / low, and between the two, with s = (original / l - low) / (high - low), becomes
+    (1 - s) f / factor + s f.  Sines and cosines keep their magnitude."""
+    factor: float
+    low: float
+    high: float
+    original: float
+
+
+@dataclass(frozen=True)
 class RotarySpec:
     """Rotation of pairs of dims by position over the first `dims` dims of a head: pair i turns by
     position * base^(-2i/dims).  Pair i is (dim i, dim i + dims/2), or with `interleaved` (dim 2i, dim 2i + 1)."""
     dims: int
     base: float
     interleaved: bool = False
-    scaling: Optional[FrequencyRampSpec] = None
+    scaling: Any = None              # FrequencyRampSpec, FrequencyBandsSpec or None
 
 
 @dataclass(frozen=True)
@@ -104,6 +116,19 @@ class RotaryAttentionSpec:
     window: Optional[int] = None
     # `v` None: there is no value projection; the values are the keys as projected (with bias), before normalisation
     # and rotation (v_dim = k_dim)
+    keep_first: int = 0              # with a window: the first keep_first positions stay visible to every later one
+    # tensors [n_heads]: distance_mul[h] * ln(1 + distance_rate[h] * (i - j)) is taken off the score (in 32-bit)
+    distance_mul: Optional[str] = None
+    distance_rate: Optional[str] = None
+    # sigmoid of its product multiplies the heads' outputs before the output projection: one number per head
+    # ([n_heads, hidden]) or, without gate_per_head, one per element ([n_heads * v_dim, hidden])
+    gate: Optional[LinearSpec] = None
+    gate_per_head: bool = False
+    # tensor []: lambda.  With value_source (the cache number of an earlier schedule entry) the values that are cached are
+    # (1 - lambda) own + lambda those projected by that entry for the same tokens; without it lambda is unused, but
+    # the projected values are kept for the entries that name this one.
+    value_mix: Optional[str] = None
+    value_source: Optional[int] = None
 
 
 @dataclass(frozen=True)
@@ -273,9 +298,35 @@ class SSDSpec:
 
 
 @dataclass(frozen=True)
+class SelectiveScanSpec:
+    """A selective state-space recurrence with a decay per channel and state ("selective scan").  The input projection's
+    rows are [x: inner | z: inner]; x passes a short causal convolution per channel (with bias) and an activation;
+    W_x x = [dt: dt_rank | B: state | C: state], dt <- softplus(W_dt dt + dt_bias) per channel; per channel c and state n
+        S[c, n] <- exp(-exp(A_log[c, n]) dt_c) S[c, n] + dt_c x_c B_n;   y_c = sum_n S[c, n] C_n + D_c x_c
+    then y * act(z) and the output projection."""
+    kind: str                        # 'selective_scan'
+    hidden: int
+    inner: int
+    state: int
+    dt_rank: int
+    conv_taps: int
+    in_proj: LinearSpec = None       # [2 inner, hidden]
+    x_proj: LinearSpec = None        # [dt_rank + 2 state, inner]
+    dt_proj: LinearSpec = None       # [inner, dt_rank]
+    out: LinearSpec = None
+    conv: str = None                 # tensor [inner, conv_taps]; the last column weighs the current token
+    conv_bias: Optional[str] = None  # tensor [inner]
+    dt_bias: str = None              # tensor [inner]
+    a_log: str = None                # tensor [inner, state]
+    skip: Optional[str] = None       # tensor [inner]: D
+    activation: str = "silu"         # of the convolution's output and of z
+
+
+@dataclass(frozen=True)
 class RetentionSpec:
     """Linear attention with a fixed decay per head: S <- decay S + k v^T, o = S^T q; each head's o divided by
-    its root mean square, gated by silu of a projection, then the output projection."""
+    its root mean square (with joint_norm: all heads' o together by theirs), times `out_norm`, gated by an activation
+    (silu) of a projection, then the output projection.  q, k and v may pass an activation behind their projections."""
     kind: str                        # 'retention'
     hidden: int
     n_heads: int
@@ -290,6 +341,10 @@ class RetentionSpec:
     rotary: Optional[RotarySpec] = None
     k_scale: float = 1.0             # keys are multiplied by it after rotation
     norm_eps: float = 1e-6
+    activation: Optional[str] = None     # of q, k and v
+    gate_activation: str = "silu"
+    joint_norm: bool = False
+    out_norm: Optional[str] = None       # tensor [v_dim], or [n_heads * v_dim] with joint_norm
 
 
 @dataclass(frozen=True)
@@ -361,6 +416,8 @@ class RoutedFeedForwardSpec:
     group_top: int = 2
     renorm_eps: float = 0.0
     weight_scale: float = 1.0
+    router_bias: Optional[str] = None    # tensor [n_experts], added to the router's logits
+    shared: Optional[GatedFeedForwardSpec] = None   # a feed-forward that every token runs, added to the chosen experts'
 
 
 @dataclass(frozen=True)

@@ -26,7 +26,7 @@ from .model_files import open_model_files
 class TensorSpec:
     name: str                      # name in the checkpoint
     shape: Tuple[int, ...]         # an entry of -1: any size (the part takes it from the stored tensor)
-    kind: str = "matrix"           # 'matrix' | 'table' | 'bias' | 'norm_weight' | 'norm_bias' | 'int_table'
+    kind: str = "matrix"           # 'matrix' | 'table' | 'bias' | 'norm_weight' | 'norm_bias' | 'positive' | 'int_table'
     tied_to: Optional[str] = None  # when absent from the file, this other tensor is used
     optional: bool = False         # may be absent without a tie (never used by OPT)
 

@@ -35,6 +35,8 @@ def random_tensors(specs: Sequence[TensorSpec], seed: int, init_std: float,
         t = torch.randn(s.shape, generator=gen, dtype=torch.float32) * init_std
         if s.kind == "norm_weight":
             out[s.name] = (1.0 + t)       # LayerNorm tensors stay in 32-bit, as the reference's
+        elif s.kind == "positive":
+            out[s.name] = t.abs().to(matrix_dtype)
         elif s.kind in ("norm_bias",):    # demo keeps them (opt/demo.py:23-29)
             out[s.name] = t
         else:
