@@ -23,6 +23,8 @@ attention whose values are its keys, attention through latents, a gated delta-ru
 closest design here (paged attention beside a recurrence with a state of fixed size), at the same widths.
 `--workload vozirax`: the Vozirax decoder (a selective state-space recurrence, differential attention with a layer that
 reads another's keys and values, gated and routed feed-forwards side by side with the mixers) beside Tutelix.
+`--workload resatar`: the Resatar decoder (attention with mixed values, windowed attention with a distance bias beside
+lightning attention, a selective scan, dense and routed feed-forwards with a shared expert) beside Vozirax.
 """
 from __future__ import annotations
 
@@ -466,6 +468,35 @@ def vozirax_config(size):
             "max_positions": CONTEXT, "layers": layers}
 
 
+# ---- the Resatar decoder beside Vozirax at equal sizes -----------------------------------------------
+# Heads of 128 dims on a quarter as many key/value heads (rotated over half their dims with stretched frequencies, the fourth
+# layer's values mixed with the first one's); a parallel layer of the same attention under a window of half the bench's
+# context that keeps its first 64 tokens, with a distance bias, beside lightning attention of as many heads of 128 x 128; a
+# selective scan of twice the width inside over a state of 16 with a step rank of W / 16 and four taps; a feed-forward of 4x
+# the width, or eight experts of which a token runs two beside a shared one, whose inner width gives a token the same parameters.
+RESATAR_SIZES = {"2048": dict(width=2048, heads=16, kv=4, ff=8192, expert_ff=1824),
+                 "4096": dict(width=4096, heads=32, kv=8, ff=16384, expert_ff=3648)}
+RESATAR_LAYERS = ("attention + dense", "parallel + moe", "mamba1 + dense", "attention + moe")
+
+
+def resatar_config(size):
+    z = RESATAR_SIZES[size]
+    W, H = z["width"], z["heads"]
+    att = {"heads": H, "kv_heads": z["kv"], "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "v_mix": True,
+           "rot": {"dims": 64, "base": 5e5, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 1024}}}
+    par = {"left": {"heads": H, "kv_heads": z["kv"], "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                    "mask": {"size": CONTEXT // 2, "keep_first": 64}},
+           "right": {"heads": H, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** (-5 - 7 * h / H) for h in range(H)]},
+           "left_scale": 1.0, "right_scale": 0.8}
+    ssm = {"inner": 2 * W, "dt_rank": W // 16, "state": 16, "conv": 4}
+    dense = {"kind": "dense", "ff": z["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": z["expert_ff"]}, "router": {"experts": 8, "top": 2}, "shared": {"ff": z["expert_ff"]}}
+    layers = [{"type": "attention", "mixer": att, "mlp": dense}, {"type": "parallel", "mixer": par, "mlp": moe},
+              {"type": "mamba1", "mixer": ssm, "mlp": dense}, {"type": "attention", "mixer": att, "mlp": moe}]
+    return {"architecture": "Resatar", "vocab": 50272, "width": W, "norm": {"eps": 1e-5}, "init_std": 0.02,
+            "max_positions": CONTEXT, "layers": layers}
+
+
 def build_vononex(size, dtype="bfloat16", config=None):
     import torch
     from transformers_neuronx_b200.config import config_from_dict
@@ -478,6 +509,7 @@ def build_vononex(size, dtype="bfloat16", config=None):
     tensors = {}
     for s in DecoderModel(spec).tensor_specs():
         t = torch.randn(s.shape, generator=g, device=dev, dtype=torch.float32) * cfg.init_std
+        t = t.abs() if s.kind == "positive" else t
         tensors[s.name] = (1.0 + t) if s.kind == "norm_weight" else t.to(getattr(torch, dtype))
     return build_model(spec, tensors, dtype, verbose=False), cfg
 
@@ -549,7 +581,13 @@ def workload_vozirax(steps, warmup, sizes=None, only=None, batch=8):
                             layers=VOZIRAX_LAYERS, config=vozirax_config, beside="tutelix")
 
 
-BESIDE_CONFIGS = {"vononex": None, "tutelix": tutelix_config}       # the designs that can stand beside another (None: Vononex's own)
+def workload_resatar(steps, warmup, sizes=None, only=None, batch=8):
+    """workload_vononex for the Resatar decoder, with Vozirax at the same width beside it."""
+    return workload_vononex(steps, warmup, sizes or ["2048", "4096"], only, batch, design="resatar", table=RESATAR_SIZES,
+                            layers=RESATAR_LAYERS, config=resatar_config, beside="vozirax")
+
+
+BESIDE_CONFIGS = {"vononex": None, "tutelix": tutelix_config, "vozirax": vozirax_config}       # the designs that can stand beside another (None: Vononex's own)
 
 
 def workload_vononex(steps, warmup, sizes=None, only=None, batch=8, design="vononex", table=None, layers=None, config=None,
@@ -612,6 +650,8 @@ def extra_workload(name, steps, warmup, sizes=None, only=None, batch=8):
         res = workload_tutelix(steps, warmup, sizes, only, batch)
     elif name == "vozirax":
         res = workload_vozirax(steps, warmup, sizes, only, batch)
+    elif name == "resatar":
+        res = workload_resatar(steps, warmup, sizes, only, batch)
     elif name == "family":
         res = workload_family(steps, warmup, sizes)
     elif name == "sweep":
@@ -647,10 +687,10 @@ def main():
     ap.add_argument("--skip-large", action="store_true", help="leave out the OPT-13B and OPT-30B workloads")
     ap.add_argument("--dtype", default="float16", choices=["float16", "bfloat16"],
                     help="the serving type (float16 is what OPT checkpoints are stored in)")
-    ap.add_argument("--workload", default=None, choices=["decode30b", "mixed13b", "family", "sweep", "vononex", "pifelix", "tutelix", "vozirax"],
+    ap.add_argument("--workload", default=None, choices=["decode30b", "mixed13b", "family", "sweep", "vononex", "pifelix", "tutelix", "vozirax", "resatar"],
                     help="run one of the further workloads instead of the default line")
     ap.add_argument("--sizes", default=None, help="for --workload family: comma-separated sizes (default: all of 125m .. 66b); for --workload vononex: "
-                    "widths (2048, 4096); for --workload tutelix: 2048, 4096, 2048wide; for --workload vozirax: 2048, 4096")
+                    "widths (2048, 4096); for --workload tutelix: 2048, 4096, 2048wide; for --workload vozirax and resatar: 2048, 4096")
     ap.add_argument("--only", default=None, choices=["decode", "prefill"],
                     help="run just this part and print its time (for profiling a small case)")
     a = ap.parse_args()

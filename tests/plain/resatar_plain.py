@@ -69,10 +69,6 @@ def rotate(x, positions, dims, base, scaling=None):
     return y
 
 
-def visible(i, j, window=None, keep=0):
-    return j <= i and (window is None or i - j < window or j < keep)
-
-
 def attend(q, k, v, scale, see, bias=None):
     """q [T, H, d], k [T, G, d], v [T, G, e], see [T, T] -> [T, H, e];  bias(h) [T, T] is taken off the scores."""
     T, H, G = q.shape[0], q.shape[1], k.shape[1]
@@ -87,11 +83,10 @@ def attend(q, k, v, scale, see, bias=None):
 
 
 def mask(T, window=None, keep=0):
-    see = torch.zeros(T, T, dtype=torch.bool)
-    for i in range(T):
-        for j in range(T):
-            see[i, j] = visible(i, j, window, keep)
-    return see
+    """[query i, key j]: j <= i, and with a window i - j < window or j among the first `keep`."""
+    i, j = torch.arange(T)[:, None], torch.arange(T)[None, :]
+    see = j <= i
+    return see if window is None else see & ((i - j < window) | (j < keep))
 
 
 def softmax_attention(h, t, p, m, first_values=None):
@@ -114,11 +109,8 @@ def softmax_attention(h, t, p, m, first_values=None):
 
 
 def distance_bias(T, r1, r2):
-    b = torch.zeros(T, T, dtype=F64)
-    for i in range(T):
-        for j in range(i + 1):
-            b[i, j] = r1 * math.log(1.0 + r2 * (i - j))
-    return b
+    d = (torch.arange(T)[:, None] - torch.arange(T)[None, :]).clamp(min=0).to(F64)
+    return r1 * torch.log(1.0 + r2 * d)
 
 
 def biased_window_attention(h, t, p, m, eps):

@@ -79,6 +79,7 @@ struct RouterOptions {
     int n_groups, keep_groups, group_top;
     float renorm_eps, weight_scale;
     const float* bias;           // [E], added to the logits, or null
+    int always;                  // further experts (E, E + 1, ...) that every token takes with weight 1, behind the chosen ones
 };
 
 template <typename T, typename TW>
@@ -94,8 +95,9 @@ moe_router_kernel(const T* __restrict__ h, int ld, const TW* __restrict__ wr, co
     pdl_launch_dependents();
     pdl_wait();
     const int n = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const size_t row = (size_t)n * (top + ro.always);        // where the token's experts and weights begin
     if (token_request[n] < 0) {                              // a padded row of a captured step: no expert
-        if (threadIdx.x < top) { ids[(size_t)n * top + threadIdx.x] = -1; weights[(size_t)n * top + threadIdx.x] = 0.f; }
+        if (threadIdx.x < top + ro.always) { ids[row + threadIdx.x] = -1; weights[row + threadIdx.x] = 0.f; }
         return;
     }
     for (int c = threadIdx.x; c < W; c += blockDim.x) x[c] = to_float(h[(size_t)n * ld + c]);
@@ -188,11 +190,13 @@ moe_router_kernel(const T* __restrict__ h, int ld, const TW* __restrict__ wr, co
         if (lane == 0) z[arg] = -INFINITY;
         __syncwarp();
     }
-    if (lane == 0)
+    if (lane == 0) {
         for (int j = 0; j < top; ++j) {
-            ids[(size_t)n * top + j] = chosen[j];
-            weights[(size_t)n * top + j] = (renormalize ? chosen_w[j] / (total + ro.renorm_eps) : chosen_w[j]) * ro.weight_scale;
+            ids[row + j] = chosen[j];
+            weights[row + j] = (renormalize ? chosen_w[j] / (total + ro.renorm_eps) : chosen_w[j]) * ro.weight_scale;
         }
+        for (int j = 0; j < ro.always; ++j) { ids[row + top + j] = E + j; weights[row + top + j] = 1.f; }
+    }
 }
 
 struct ExpertMath {
@@ -432,14 +436,15 @@ moe_sum_kernel(const float* __restrict__ per_pair, const int* __restrict__ ids, 
 TNX_EXPORT int tnx_moe_route(const void* h, int ld, const void* router, const int* token_request, int* ids, float* weights,
                              int N, int W, int E, int top, int softmax_scores, int renormalize, int h_h16, int w_h16,
                              const float* correction, int n_groups, int keep_groups, int group_top, float renorm_eps,
-                             float weight_scale, const float* bias, cudaStream_t stream) {
+                             float weight_scale, const float* bias, int always, cudaStream_t stream) {
     if (N <= 0) return 0;
     if (W <= 0 || E <= 0 || E > MAX_EXPERTS || top <= 0 || top > MAX_TOP || top > E) return TNX_ERR_UNSUPPORTED;
+    if (always < 0 || top + always > MAX_TOP || E + always > MAX_EXPERTS) return TNX_ERR_UNSUPPORTED;
     if (n_groups < 1 || E % n_groups || keep_groups < 1 || keep_groups > n_groups || group_top < 1 ||
         (long long)keep_groups * (E / n_groups) < top || ((correction || n_groups > 1) && softmax_scores))
         return TNX_ERR_BAD_ARG;
     if (n_groups > 1 && E / n_groups > 64 && group_top > 1) return TNX_ERR_UNSUPPORTED;
-    const RouterOptions ro{correction, n_groups, keep_groups, group_top, renorm_eps, weight_scale, bias};
+    const RouterOptions ro{correction, n_groups, keep_groups, group_top, renorm_eps, weight_scale, bias, always};
     const size_t smem = (size_t)(((W + 3) & ~3) + 3 * E) * sizeof(float);
     if (smem > 160 * 1024) return TNX_ERR_UNSUPPORTED;
 #define GO(T, TW)                                                                                                       \

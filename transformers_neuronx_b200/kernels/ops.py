@@ -91,7 +91,7 @@ _FLOATS = (torch.float32,) + _H16
 # Activations a product's epilogue applies, by the names the reference looks up
 # (src/transformers_neuronx/hlo.py:485-501 -> activations.py) -> the kernels' codes (csrc/common.cuh).
 ACTIVATIONS = {None: 0, "none": 0, "relu": 1, "gelu_new": 2, "gelu_new_legacy": 2, "gelu_pytorch_tanh": 2,
-               "silu": 3, "swish": 3, "sigmoid": 4, "gelu": 5}
+               "silu": 3, "swish": 3, "sigmoid": 4, "gelu": 5, "softplus": 6}
 
 
 def activation_code(name) -> int:
@@ -974,13 +974,15 @@ def conv_qkv_prep(proj, col0, conv_w, taps, state, ctx, q_norm, k_norm, eps, inv
 
 
 def moe_route(h, router, token_request, ids, weights, top, softmax_scores=False, renormalize=False, correction=None,
-              n_groups=1, keep_groups=1, group_top=2, renorm_eps=0.0, weight_scale=1.0, bias=None):
+              n_groups=1, keep_groups=1, group_top=2, renorm_eps=0.0, weight_scale=1.0, bias=None,
+              always=0):
     """For every row of h [N, W]: the `top` experts with the largest scores (sigmoid, or softmax, of the 32-bit product
     with router [E, W], plus bias [E] where it is given) into ids [N, top] (int32; -1 for a padded row) and their scores into weights [N, top].
     correction (32-bit [E]): added to the sigmoid scores for the choice only.  n_groups > 1: the experts form equal groups
     of neighbours, a group's score is the sum of its group_top largest choice scores, and only experts of the keep_groups
     best groups can be chosen.  The weights are divided by (their sum + renorm_eps) with `renormalize`, then multiplied
-    by weight_scale."""
+    by weight_scale.  always: as many further experts (E, E + 1, ...), with weight 1 each, stand behind the chosen ones in
+    every row (ids and weights are then [N, top + always])."""
     lib = _lib("moe", h, router)
     _need(h, "h", _FLOATS, None, contiguous=False)
     N, W, ld = _rows_2d(h, "h")
@@ -990,13 +992,13 @@ def moe_route(h, router, token_request, ids, weights, top, softmax_scores=False,
         raise KernelError("the router's rows must be as long as h's")
     _need(token_request, "token_request", torch.int32, 1)
     _need(ids, "ids", torch.int32, 2); _need(weights, "weights", torch.float32, 2)
-    if tuple(ids.shape) != (N, top) or tuple(weights.shape) != (N, top):
-        raise KernelError(f"ids and weights must be [{N}, {top}]")
+    if tuple(ids.shape) != (N, top + always) or tuple(weights.shape) != (N, top + always):
+        raise KernelError(f"ids and weights must be [{N}, {top + always}]")
     _f32_vec(correction, "correction", E); _f32_vec(bias, "bias", E)
     _check(lib.tnx_moe_route(_p(h), c_int(ld), _p(router), _p(token_request), _p(ids), _p(weights), c_int(N), c_int(W),
                              c_int(E), c_int(top), c_int(1 if softmax_scores else 0), c_int(1 if renormalize else 0),
                              c_int(_is_h16(h)), c_int(_is_h16(router)), _p(correction), c_int(n_groups), c_int(keep_groups),
-                             c_int(group_top), c_float(renorm_eps), c_float(weight_scale), _p(bias), _stream()), "moe_route")
+                             c_int(group_top), c_float(renorm_eps), c_float(weight_scale), _p(bias), c_int(always), _stream()), "moe_route")
 
 
 EXPERT_FORMS = {"gated_swish": 0, "relu2": 1}
@@ -1476,8 +1478,8 @@ def causal_conv(proj, col0, conv_w, conv_b, taps, state, ctx, activation, out):
         conv_state_update(proj, col0, state, ctx)
 
 
-def selective_scan(x, dt, low, b_off, c_off, decay_log2, dt_bias, skip, z, state, ctx, activation, out):
-    """Per channel c and state n, token by token for every request of the step: dt <- softplus(dt + dt_bias),
+def selective_scan(x, dt, low, b_off, c_off, decay_log2, skip, z, state, ctx, activation, out):
+    """Per channel c and state n, token by token for every request of the step:
     S[c, n] <- 2^(decay_log2[c, n] dt_c) S[c, n] + dt_c x_c B_n, out_c = (sum_n S[c, n] C_n + skip_c x_c) * act(z_c).
     x, z, out: views [N, C] in the activation type; dt 32-bit [N, C]; B and C the state-many columns of `low` at b_off and
     c_off; state 32-bit [slots, C, n], decay_log2 32-bit [C, n]."""
@@ -1496,14 +1498,21 @@ def selective_scan(x, dt, low, b_off, c_off, decay_log2, dt_bias, skip, z, state
     if dt.shape[1] != C or tuple(decay_log2.shape) != (C, Ns) or max(b_off, c_off) + Ns > low.shape[1] or min(b_off, c_off) < 0:
         raise KernelError("dt, decay_log2 or low do not fit the state's channels")
     _need(decay_log2, "decay_log2", torch.float32, 2)
-    _f32_vec(dt_bias, "dt_bias", C); _f32_vec(skip, "skip", C)
+    _f32_vec(skip, "skip", C)
     for t, nm in ((ctx.q_start, "q_start"), (ctx.q_len, "q_len"), (ctx.state_slots, "state_slots")):
         _need(t, nm, torch.int32, 1)
     _check(lib.tnx_selective_scan(_p(x), c_int(lds[0]), _p(dt), _p(low), c_int(lds[3]), c_int(b_off), c_int(c_off),
-                                  _p(decay_log2), _p(dt_bias), _p(skip), _p(z), c_int(lds[1]), _p(state), _p(ctx.q_start),
+                                  _p(decay_log2), _p(skip), _p(z), c_int(lds[1]), _p(state), _p(ctx.q_start),
                                   _p(ctx.q_len), _p(ctx.state_slots), c_int(activation_code(activation)), _p(out),
                                   c_int(lds[2]), c_int(ctx.q_len.shape[0]), c_int(C), c_int(Ns),
                                   c_int(1 if ctx.decode_only else N), c_int(_is_h16(x)), _stream()), "selective_scan")
+
+
+def selective_scan_force(states=0, dtype=None) -> None:
+    """A test and measurement hook: how many states of a channel a lane keeps (0: the kernel's own choice; 2 or 4)."""
+    lib = _build.load("selective_scan", dtype if dtype in _H16 else None)
+    if lib.tnx_selective_scan_force(c_int(int(states))) != 0:
+        raise KernelError(f"selective_scan_force: {states} states a lane is not a choice")
 
 
 def diff_qkv_prep(proj, col0, token_request, positions, q_norm, k_norm, eps, temp_coef, temp_every, q_out, k_out, v_out,

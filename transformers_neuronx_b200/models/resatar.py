@@ -52,8 +52,8 @@ def _selective_scan(p: str, W: int, m: dict) -> SelectiveScanSpec:
     C, R, N = m["inner"], m["dt_rank"], m["state"]
     return SelectiveScanSpec(kind="selective_scan", hidden=W, inner=C, state=N, dt_rank=R, conv_taps=m["conv"],
                              in_proj=_lin(p + ".in", W, 2 * C), x_proj=_lin(p + ".x", C, R + 2 * N),
-                             dt_proj=_lin(p + ".dt", R, C), out=_lin(p + ".o", C, W), conv=p + ".conv",
-                             conv_bias=p + ".conv.b", dt_bias=p + ".dt.b", a_log=p + ".A_log", skip=p + ".D",
+                             dt_proj=_lin(p + ".dt", R, C, True), out=_lin(p + ".o", C, W), conv=p + ".conv",
+                             conv_bias=p + ".conv.b", a_log=p + ".A_log", skip=p + ".D",
                              activation="silu")
 
 

@@ -9,6 +9,9 @@ to the best groups of experts, and scale the weights: parts/spec.py: RoutedFeedF
   result = sum_j expert_{e_j}(w_j h)  (weight_on_input)   or   sum_j w_j expert_{e_j}(h)
            (+ shared(h), a gated feed-forward that every token runs)
 
+A shared feed-forward of the experts' own form and inner width is one more expert that every token takes with weight 1: it
+rides in the experts' products.  Any other runs as the gated feed-forward it is, behind them.
+
 The experts' matrices are kept stacked, [E, 2 ff, hidden] (gate rows, then up rows) and [E, hidden, ff], in the type
 they are stored in.  A step routes on the device (no read on the host: the part is graph-safe) and then takes one of
 two forms: in a 16-bit engine the (token, expert) pairs are sorted by expert and run as grouped products on the tensor
@@ -25,7 +28,7 @@ from ..kernels import ops
 from ..weights.loader import TensorSpec
 from .base import FeedForward, to_device, weight_to_device
 from .registry import build_part, register_feed_forward
-from .spec import RoutedFeedForwardSpec
+from .spec import ExpertSpec, RoutedFeedForwardSpec
 
 
 class RoutedExperts(FeedForward):
@@ -34,7 +37,7 @@ class RoutedExperts(FeedForward):
 
     @property
     def libraries(self):
-        return ("moe", "moe_grouped", "gemm_tc") + (tuple(self.shared.libraries) if self.shared is not None else ())
+        return ("moe", "moe_grouped", "gemm_tc") + (tuple(self.shared.libraries) if self.shared is not None and not self.folded else ())
 
     # Rows from which the grouped tensor-core form runs in a 16-bit engine.  Measured at width 2048 (8 experts of inner
     # width 2816, 2 a token): a decode step of 1 / 8 / 32 requests takes 0.48 / 0.75 / 1.03 ms with it and 0.52 / 1.10 /
@@ -61,6 +64,11 @@ class RoutedExperts(FeedForward):
         if (s.correction or s.n_groups > 1) and s.scores != "sigmoid":
             raise ValueError("a correction of the choice and groups of experts go with sigmoid scores")
         self.shared = build_part("feed_forward", s.shared)
+        sh = s.shared
+        self.folded = (sh is not None and self.gated and sh.activation == "silu" and sh.up.out_features == s.ff
+                       and not (sh.gate.bias or sh.up.bias or sh.down.bias) and s.act_alpha == 1.0 and s.up_shift == 0.0
+                       and s.gate_limit is None and s.up_limit is None and not s.weight_on_input
+                       and s.top < 16 and s.n_experts < 1024)
         self.router = self.gate_up = self.down = self.correction = self.router_bias = None
 
     def tensor_specs(self):
@@ -83,13 +91,16 @@ class RoutedExperts(FeedForward):
             self.correction = to_device(tensors[s.correction], device, torch.float32)
         if s.router_bias:
             self.router_bias = to_device(tensors[s.router_bias], device, torch.float32)
-        if self.shared is not None:
+        if self.shared is not None and not self.folded:
             self.shared.load(tensors, device, act_dtype)
         first = weight_to_device(tensors[s.experts[0].up], device, act_dtype, s.experts[0].up)
         # gate rows, then up rows; experts without a gate: the up rows alone
-        self.gate_up = torch.empty((s.n_experts, (2 if self.gated else 1) * s.ff, s.hidden), dtype=first.dtype, device=device)
-        self.down = torch.empty((s.n_experts, s.hidden, s.ff), dtype=first.dtype, device=device)
-        for i, e in enumerate(s.experts):
+        experts = s.experts
+        if self.folded:
+            experts += (ExpertSpec(s.shared.gate.weight, s.shared.up.weight, s.shared.down.weight),)
+        self.gate_up = torch.empty((len(experts), (2 if self.gated else 1) * s.ff, s.hidden), dtype=first.dtype, device=device)
+        self.down = torch.empty((len(experts), s.hidden, s.ff), dtype=first.dtype, device=device)
+        for i, e in enumerate(experts):
             mats = ((e.gate, self.gate_up[i, :s.ff]), (e.up, self.gate_up[i, s.ff:]), (e.down, self.down[i])) if self.gated \
                 else ((e.up, self.gate_up[i]), (e.down, self.down[i]))
             for name, dst in mats:
@@ -100,7 +111,7 @@ class RoutedExperts(FeedForward):
 
     def parameter_bytes(self):
         return sum(t.numel() * t.element_size() for t in (self.router, self.gate_up, self.down, self.correction, self.router_bias)
-                   if t is not None) + (self.shared.parameter_bytes() if self.shared is not None else 0)
+                   if t is not None) + (self.shared.parameter_bytes() if self.shared is not None and not self.folded else 0)
 
     def step_bytes(self, n_tokens: int) -> int:
         """Bytes of weights a step of n_tokens is expected to read: every expert once that some token chooses, with
@@ -108,16 +119,17 @@ class RoutedExperts(FeedForward):
         s = self.spec
         used = s.n_experts * (1.0 - (1.0 - s.top / s.n_experts) ** n_tokens)
         per = (self.gate_up[0].numel() + self.down[0].numel()) * self.gate_up.element_size()
-        return int(self.router.numel() * self.router.element_size() + used * per) + \
-            (self.shared.parameter_bytes() if self.shared is not None else 0)
+        shared = 0 if self.shared is None else (per if self.folded else self.shared.parameter_bytes())
+        return int(self.router.numel() * self.router.element_size() + used * per) + shared
 
     def forward(self, ctx, h, out, accumulate=True):
         s, N = self.spec, h.shape[0]
-        ids = ctx.scratch(N, s.top, torch.int32)
-        weights = ctx.scratch(N, s.top, torch.float32)
+        always = 1 if self.folded else 0
+        ids = ctx.scratch(N, s.top + always, torch.int32)
+        weights = ctx.scratch(N, s.top + always, torch.float32)
         ops.moe_route(h, self.router, ctx.token_request, ids, weights, s.top, softmax_scores=s.scores == "softmax",
                       renormalize=s.renormalize, correction=self.correction, n_groups=s.n_groups, keep_groups=s.keep_groups,
-                      group_top=s.group_top, renorm_eps=s.renorm_eps, weight_scale=s.weight_scale, bias=self.router_bias)
+                      group_top=s.group_top, renorm_eps=s.renorm_eps, weight_scale=s.weight_scale, bias=self.router_bias, always=always)
         inf = math.inf
         limits = (s.gate_limit if s.gate_limit is not None else inf, -s.up_limit if s.up_limit is not None else -inf,
                   s.up_limit if s.up_limit is not None else inf)
@@ -125,11 +137,12 @@ class RoutedExperts(FeedForward):
             ops.moe_grouped(ctx, h, self.gate_up, self.down, ids, weights, out, *limits, s.act_alpha, s.up_shift,
                             weight_on_input=s.weight_on_input, accumulate=accumulate, form=s.expert_form)
         else:
-            y = ctx.scratch(N * s.top, s.ff)
+            pairs = N * (s.top + always)
+            y = ctx.scratch(pairs, s.ff)
             ops.moe_experts(h, self.gate_up, self.down, ids, weights, y, out, *limits, s.act_alpha, s.up_shift,
                             weight_on_input=s.weight_on_input, accumulate=accumulate,
-                            per_pair=ctx.scratch(N * s.top, s.hidden, torch.float32), form=s.expert_form)
-        if self.shared is not None:
+                            per_pair=ctx.scratch(pairs, s.hidden, torch.float32), form=s.expert_form)
+        if self.shared is not None and not self.folded:
             self.shared.forward(ctx, h, out)
 
 

@@ -9,7 +9,7 @@
 What the mixer keeps per request, both state of fixed size in the request's slot (zeroed when a request takes it): S
 (inner x state) in 32-bit, and the last taps - 1 projected values of every convolved channel in the activation type, exactly
 what a longer step would have read from its own rows.  Products and the convolution with its activation are in the
-activation type, except that W_dt's product stays 32-bit; softplus, decays, state and y are 32-bit.  A step's tokens of
+activation type, except that W_dt's product stays 32-bit (bias and softplus in its epilogue); decays, state and y are 32-bit.  A step's tokens of
 one request are walked in order by one kernel, portions of prompts and single tokens alike, so the state after a token does
 not depend on how the prompt was cut.
 """
@@ -47,7 +47,7 @@ class SelectiveScan(Mixer):
         activation_code(s.activation)
         self.keep = s.conv_taps - 1
         self.in_proj, self.x_proj, self.dt_proj, self.out = (Linear(p) for p in (s.in_proj, s.x_proj, s.dt_proj, s.out))
-        self.conv_w = self.conv_b = self.decay_log2 = self.dt_bias = self.skip = None
+        self.conv_w = self.conv_b = self.decay_log2 = self.skip = None
 
     def tensor_specs(self):
         s = self.spec
@@ -57,7 +57,7 @@ class SelectiveScan(Mixer):
         out.append(TensorSpec(s.conv, (s.inner, s.conv_taps), "matrix"))
         if s.conv_bias:
             out.append(TensorSpec(s.conv_bias, (s.inner,), "bias"))
-        out += [TensorSpec(s.dt_bias, (s.inner,), "bias"), TensorSpec(s.a_log, (s.inner, s.state), "matrix")]
+        out += [TensorSpec(s.a_log, (s.inner, s.state), "matrix")]
         if s.skip:
             out.append(TensorSpec(s.skip, (s.inner,), "bias"))
         return out
@@ -68,13 +68,13 @@ class SelectiveScan(Mixer):
             p.load(tensors, device, act_dtype)
         f32 = lambda name: to_device(tensors[name], device, torch.float32) if name else None
         self.conv_w = f32(s.conv).t().contiguous()            # [taps, channels]: a tap's weights of consecutive channels together
-        self.conv_b, self.dt_bias, self.skip = f32(s.conv_bias), f32(s.dt_bias), f32(s.skip)
+        self.conv_b, self.skip = f32(s.conv_bias), f32(s.skip)
         # the kernel's decay is 2^(decay_log2 * dt)
         self.decay_log2 = (-torch.exp(tensors[s.a_log].to(torch.float64)) / math.log(2.0)).to(torch.float32).to(device)
 
     def parameter_bytes(self):
         n = sum(p.parameter_bytes() for p in (self.in_proj, self.x_proj, self.dt_proj, self.out))
-        return n + sum(t.numel() * 4 for t in (self.conv_w, self.conv_b, self.decay_log2, self.dt_bias, self.skip) if t is not None)
+        return n + sum(t.numel() * 4 for t in (self.conv_w, self.conv_b, self.decay_log2, self.skip) if t is not None)
 
     def cache_need(self):
         s = self.spec
@@ -93,9 +93,9 @@ class SelectiveScan(Mixer):
         low = pitched(ctx, N, R + 2 * Ns)
         self.x_proj.forward(x, low)
         dt = ctx.scratch(N, C, torch.float32)
-        self.dt_proj.forward(low[:, :R], dt)
+        self.dt_proj.forward(low[:, :R], dt, activation="softplus")
         y = ctx.scratch(N, C)
-        ops.selective_scan(x, dt, low, R, R + Ns, self.decay_log2, self.dt_bias, self.skip, proj[:, C:2 * C], ctx.cache(0), ctx,
+        ops.selective_scan(x, dt, low, R, R + Ns, self.decay_log2, self.skip, proj[:, C:2 * C], ctx.cache(0), ctx,
                            s.activation, y)
         self.out.forward(y, out, residual=out if accumulate else None)
 

@@ -312,11 +312,10 @@ class SelectiveScanSpec:
     conv_taps: int
     in_proj: LinearSpec = None       # [2 inner, hidden]
     x_proj: LinearSpec = None        # [dt_rank + 2 state, inner]
-    dt_proj: LinearSpec = None       # [inner, dt_rank]
+    dt_proj: LinearSpec = None       # [inner, dt_rank]; its bias is dt_bias
     out: LinearSpec = None
     conv: str = None                 # tensor [inner, conv_taps]; the last column weighs the current token
     conv_bias: Optional[str] = None  # tensor [inner]
-    dt_bias: str = None              # tensor [inner]
     a_log: str = None                # tensor [inner, state]
     skip: Optional[str] = None       # tensor [inner]: D
     activation: str = "silu"         # of the convolution's output and of z
