@@ -264,7 +264,7 @@ def _walk(seqs, slots, cuts_list, step):
     (24, 4, 200, 3, 0, torch.float32), (72, 8, 6, 4, 4, torch.float32), (256, 16, 16, 4, 0, torch.bfloat16)])
 def test_the_selective_scan_across_cuts_and_slots(C, R, N, taps, states, dtype):
     """Two requests cut into unequal steps side by side (single tokens, pairs, a padded row, a request left out of a step):
-    convolution with bias and silu, decays per channel and state, skip and gate, against the plain recurrence over the whole
+    convolution with bias and silu, step sizes, decays per channel and state, skip and gate, against the plain recurrence over the whole
     sequences; a slot nobody uses stays as it is, and a request that takes a freed (zeroed) slot does not see what was there."""
     from transformers_neuronx_b200.kernels import ops
     g = torch.Generator().manual_seed(5)
@@ -294,12 +294,12 @@ def test_the_selective_scan_across_cuts_and_slots(C, R, N, taps, states, dtype):
         x = RP.silu(RP.causal_conv(s[:, :C], w.double(), b.double()))
         if dtype == torch.bfloat16:
             x = x.bfloat16().double()
-        y, S = RP.scan(x, s[:, -C:], -torch.exp(a_log.double()), s[:, 2 * C + R:2 * C + R + N], s[:, 2 * C + R + N:2 * C + R + 2 * N], D.double())
+        y, S = RP.scan(x, torch.nn.functional.softplus(s[:, -C:], threshold=1e9), -torch.exp(a_log.double()), s[:, 2 * C + R:2 * C + R + N], s[:, 2 * C + R + N:2 * C + R + 2 * N], D.double())
         return torch.cat([x, y * RP.silu(s[:, C:2 * C])], 1), S
 
     seqs = []
     for _ in range(3):
-        s = torch.cat([rnd(T, 2 * C + R + 2 * N).to(dtype).float(), torch.nn.functional.softplus(rnd(T, C) - 1.0)], 1)
+        s = torch.cat([rnd(T, 2 * C + R + 2 * N).to(dtype).float(), rnd(T, C) * 3 - 1.0], 1)          # step sizes before their softplus
         seqs.append(s)
     ops.selective_scan_force(states, dtype)
     try:
@@ -410,20 +410,24 @@ def test_experts_with_a_shared_one(E, top, ff, shared, W, N, dtype):
         ctx.begin_entry()
 
 
-def test_the_step_sizes_epilogue():
-    """softplus behind a product, in 32-bit, from the far negative side to where it is the identity."""
+@pytest.mark.parametrize("N, K, F", [(300, 128, 512), (130, 72, 88), (5, 256, 512), (1, 256, 512), (2048, 64, 1000)])
+def test_gelu_behind_the_up_product(N, K, F):
+    """The tanh form of gelu in the products' epilogues (whole tiles, ragged edges, few tokens), over inputs from far below to
+    far above zero; results are 16-bit."""
     from transformers_neuronx_b200.parts.linear import Linear
     from transformers_neuronx_b200.parts.spec import LinearSpec
-    for dtype in (torch.float32, torch.bfloat16):
-        lin = Linear(LinearSpec(16, 40, "w", "b"))
-        b = torch.linspace(-30, 40, 40)
-        w = (torch.randn(40, 16, generator=torch.Generator().manual_seed(9)) * 0.2).to(dtype)
-        lin.load({"w": w, "b": b}, torch.device(DEV), dtype)
-        a = torch.randn(33, 16, generator=torch.Generator().manual_seed(10)).to(dtype)
-        out = torch.empty(33, 40, device=DEV)
-        lin.forward(a.to(DEV), out, activation="softplus")
-        want = torch.nn.functional.softplus(a.double() @ w.double().T + b.double(), threshold=1e9)
-        assert float(((out.cpu().double() - want).abs() / want).max()) <= (3e-6 if dtype == torch.float32 else 2e-5)
+    g = torch.Generator().manual_seed(9)
+    for dtype in (torch.bfloat16, torch.float32):
+        lin = Linear(LinearSpec(K, F, "w"))
+        w = (torch.randn(F, K, generator=g) * torch.logspace(-2, 0, F)[:, None]).to(dtype)
+        lin.load({"w": w}, torch.device(DEV), dtype)
+        a = torch.randn(N, K, generator=g).to(dtype)
+        out = torch.empty(N, F, device=DEV, dtype=dtype)
+        lin.forward(a.to(DEV), out, activation="gelu_new")
+        want = RP.gelu_tanh(a.double() @ w.double().T)
+        err = (out.cpu().double() - want).abs()
+        tol = 2e-6 if dtype == torch.float32 else 2.0 ** -8
+        assert float((err - tol * want.abs()).max()) <= (2e-5 if dtype == torch.float32 else 1e-4)
 
 
 # ---- whole models through the replay program's function -------------------------------------------

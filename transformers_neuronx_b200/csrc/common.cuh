@@ -108,7 +108,7 @@ template <> __device__ __forceinline__ h16 from_float<h16>(float v) { return flo
 
 // Activations that a product's epilogue applies to (sum + bias), by code: the names of
 // src/transformers_neuronx/activations.py (relu :43-48, gelu_new :17-41 with its tanh form, sigmoid
-// :66-67, silu :70-72) plus the exact (erf) gelu and the softplus of a recurrence's step sizes.  The code travels to the kernel as a number, so
+// :66-67, silu :70-72) plus the exact (erf) gelu.  The code travels to the kernel as a number, so
 // another activation is one more case here and one more name in kernels/ops.py.
 #define TNX_ACT_NONE 0
 #define TNX_ACT_RELU 1
@@ -116,8 +116,7 @@ template <> __device__ __forceinline__ h16 from_float<h16>(float v) { return flo
 #define TNX_ACT_SILU 3
 #define TNX_ACT_SIGMOID 4
 #define TNX_ACT_GELU 5
-#define TNX_ACT_SOFTPLUS 6
-#define TNX_ACT_COUNT 7
+#define TNX_ACT_COUNT 6
 // The two cheap cases are inline; everything else is one call into a function that is compiled once.
 // (With every case expanded inline, the epilogues of the tensor-core products, which apply the
 // activation to several accumulators per loop turn, grew so much that a 2,048-token prefill of the
@@ -127,10 +126,15 @@ __device__ __noinline__ float apply_activation_other(float v, int act) {
         case TNX_ACT_GELU_NEW: return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
         case TNX_ACT_SILU: return v / (1.f + expf(-v));
         case TNX_ACT_SIGMOID: return 1.f / (1.f + expf(-v));
-        case TNX_ACT_SOFTPLUS: return v > 20.f ? v : log1pf(expf(v));
         case TNX_ACT_GELU: return 0.5f * v * (1.f + erff(v * 0.7071067811865476f));
         default: return v;
     }
+}
+// The tanh form of gelu for epilogues that round to 16 bits anyway and meet it by the million: 0.5 (1 + tanh u) is
+// 1 / (1 + e^(-2u)), a handful of instructions that stay inline.
+__device__ __forceinline__ float gelu_new_fast(float v) {
+    const float u2 = fmaxf(1.5957691216057308f * (v + 0.044715f * v * v * v), -80.f);
+    return __fdividef(v, 1.f + __expf(-u2));
 }
 // Eight neighbouring channels as one 16-byte access (two for floats), and as floats.
 template <typename T> struct Vec8;

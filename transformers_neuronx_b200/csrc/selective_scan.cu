@@ -1,8 +1,8 @@
 // A selective state-space recurrence with a decay per channel and state ("selective scan").  Per channel c and state n:
+//     dt_c <- softplus(dt_c)
 //     S[c, n] <- 2^(decay_log2[c, n] dt_c) S[c, n] + dt_c x_c B_n          (S: 32-bit, kept per request between steps)
 //     out_c = (sum_n S[c, n] C_n + skip_c x_c) * act(z_c)
-// with decay_log2 = -exp(A_log) log2(e) and step sizes dt as they come (the product in front has applied bias and softplus);
-// B and C of a token are shared by all channels.
+// with decay_log2 = -exp(A_log) log2(e); B and C of a token are shared by all channels.
 //
 // tnx_causal_conv: one short causal convolution per channel over a request's tokens, with bias and activation,
 //     y_t[c] = act(bias[c] + sum_j w[j, c] u_(t - taps + 1 + j)[c])       (zeros before position 0; the past comes from
@@ -24,6 +24,7 @@ namespace {
 constexpr int MAX_TAPS = 8;
 constexpr int THREADS = 128;
 
+__device__ __forceinline__ float softplus_f(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 __device__ __forceinline__ float exp2_approx(float x) {
     float y;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
@@ -238,7 +239,7 @@ __global__ void __launch_bounds__(THREADS) selective_scan_kernel(const ScanArgs<
 #pragma unroll
         for (int i = 0; i < XN; ++i) {
             const int t = tk + i * STEP;
-            const float dt = t0 + t < len ? r_dt[i] : 0.f;
+            const float dt = t0 + t < len ? softplus_f(r_dt[i]) : 0.f;
             if (XN * STEP == ST || t < ST) {
                 dts[s][ck][t] = dt;
                 dtx[s][ck][t] = dt * to_float(r_x[i]);
@@ -342,7 +343,7 @@ __global__ void __launch_bounds__(THREADS) selective_step_kernel(const ScanArgs<
     float* st = p.state + ((size_t)slot * C + cc) * Ns;
     load_states<SPT>(st, n0, Ns, mine, S);
     load_states<SPT>(p.decay_log2 + (size_t)cc * Ns, n0, Ns, mine, a2);
-    const float d = p.dt[n * C + cc], x = to_float(p.x[n * p.x_ld + cc]), z = to_float(p.z[n * p.z_ld + cc]);
+    const float d = softplus_f(p.dt[n * C + cc]), x = to_float(p.x[n * p.x_ld + cc]), z = to_float(p.z[n * p.z_ld + cc]);
     const T* low = p.low + n * p.low_ld;
     const float w = d * x;
     float y = 0.f;

@@ -91,7 +91,7 @@ _FLOATS = (torch.float32,) + _H16
 # Activations a product's epilogue applies, by the names the reference looks up
 # (src/transformers_neuronx/hlo.py:485-501 -> activations.py) -> the kernels' codes (csrc/common.cuh).
 ACTIVATIONS = {None: 0, "none": 0, "relu": 1, "gelu_new": 2, "gelu_new_legacy": 2, "gelu_pytorch_tanh": 2,
-               "silu": 3, "swish": 3, "sigmoid": 4, "gelu": 5, "softplus": 6}
+               "silu": 3, "swish": 3, "sigmoid": 4, "gelu": 5}
 
 
 def activation_code(name) -> int:
@@ -1479,7 +1479,7 @@ def causal_conv(proj, col0, conv_w, conv_b, taps, state, ctx, activation, out):
 
 
 def selective_scan(x, dt, low, b_off, c_off, decay_log2, skip, z, state, ctx, activation, out):
-    """Per channel c and state n, token by token for every request of the step:
+    """Per channel c and state n, token by token for every request of the step: dt <- softplus(dt),
     S[c, n] <- 2^(decay_log2[c, n] dt_c) S[c, n] + dt_c x_c B_n, out_c = (sum_n S[c, n] C_n + skip_c x_c) * act(z_c).
     x, z, out: views [N, C] in the activation type; dt 32-bit [N, C]; B and C the state-many columns of `low` at b_off and
     c_off; state 32-bit [slots, C, n], decay_log2 32-bit [C, n]."""

@@ -9,7 +9,7 @@
 What the mixer keeps per request, both state of fixed size in the request's slot (zeroed when a request takes it): S
 (inner x state) in 32-bit, and the last taps - 1 projected values of every convolved channel in the activation type, exactly
 what a longer step would have read from its own rows.  Products and the convolution with its activation are in the
-activation type, except that W_dt's product stays 32-bit (bias and softplus in its epilogue); decays, state and y are 32-bit.  A step's tokens of
+activation type, except that W_dt's product (with its bias) stays 32-bit; softplus, decays, state and y are 32-bit.  A step's tokens of
 one request are walked in order by one kernel, portions of prompts and single tokens alike, so the state after a token does
 not depend on how the prompt was cut.
 """
@@ -93,7 +93,7 @@ class SelectiveScan(Mixer):
         low = pitched(ctx, N, R + 2 * Ns)
         self.x_proj.forward(x, low)
         dt = ctx.scratch(N, C, torch.float32)
-        self.dt_proj.forward(low[:, :R], dt, activation="softplus")
+        self.dt_proj.forward(low[:, :R], dt)
         y = ctx.scratch(N, C)
         ops.selective_scan(x, dt, low, R, R + Ns, self.decay_log2, self.skip, proj[:, C:2 * C], ctx.cache(0), ctx,
                            s.activation, y)
