@@ -24,7 +24,16 @@ namespace {
 constexpr int MAX_TAPS = 8;
 constexpr int THREADS = 128;
 
-__device__ __forceinline__ float softplus_f(float x) { return x > 20.f ? x : log1pf(expf(x)); }
+// softplus(x) = max(x, 0) + ln(1 + e), e = exp(-|x|), and ln(1 + e) = 2 artanh(r), r = e / (2 + e) <= 1/3, by its power series
+// r + r^3/3 + r^5/5 + ...: exact to a few units of the last place for tiny e as well, and without a branch, so that a
+// thread's several step sizes are formed together.
+__device__ __forceinline__ float softplus_f(float x) {
+    const float e = __expf(-fabsf(x)), r = __fdividef(e, 2.f + e), q = r * r;
+    float t = 1.f / 15.f;
+    t = fmaf(t, q, 1.f / 13.f); t = fmaf(t, q, 1.f / 11.f); t = fmaf(t, q, 1.f / 9.f);
+    t = fmaf(t, q, 1.f / 7.f); t = fmaf(t, q, 1.f / 5.f); t = fmaf(t, q, 1.f / 3.f);
+    return fmaxf(x, 0.f) + 2.f * fmaf(t * q, r, r);
+}
 __device__ __forceinline__ float exp2_approx(float x) {
     float y;
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
@@ -32,7 +41,7 @@ __device__ __forceinline__ float exp2_approx(float x) {
 }
 // the activation the design uses inline, any other by the common function
 __device__ __forceinline__ float act_inline(float v, int act) {
-    return act == TNX_ACT_SILU ? v / (1.f + expf(-v)) : apply_activation(v, act);
+    return act == TNX_ACT_SILU ? __fdividef(v, 1.f + __expf(-v)) : apply_activation(v, act);
 }
 
 template <typename T>
@@ -376,13 +385,14 @@ int g_force_states = 0;
 
 template <typename T>
 int scan_by_state(const ScanArgs<T>& p, int n_requests, int most_tokens, cudaStream_t stream) {
-    // Two states a lane make twice the warps of half the work a token: faster where four leave the SMs fewer than one and a
-    // half blocks each.  Measured, 2,048 tokens over a state of 16: 2,048 channels 197 us with four and 141 with two states a
-    // lane, 4,096 channels 197 and 165, 8,192 channels 231 and 225; four requests of 512 tokens of 4,096 channels 94 and 97.
+    // Two states a lane make twice the warps of half the work a token: faster where four leave the SMs fewer than two blocks
+    // each (one, for states above 16).  Measured, 2,048 tokens over a state of 16: 2,048 channels 219 us with four and 160
+    // with two states a lane, 4,096 channels 221 and 178, 8,192 channels 254 and 239; four requests of 512 tokens of 4,096
+    // channels 98 and 101; 4,096 channels over a state of 32 210 and 223.
     static int sms = 0;
     if (!sms) { int dev = 0; cudaGetDevice(&dev); cudaDeviceGetAttribute(&sms, cudaDevAttrMultiProcessorCount, dev); if (sms <= 0) sms = 1; }
     const long long lanes = (long long)p.C * ((p.Ns + 3) / 4) * n_requests;
-    const int spt = g_force_states ? g_force_states : (2 * lanes < 3LL * sms * THREADS ? 2 : 4);
+    const int spt = g_force_states ? g_force_states : (lanes < (p.Ns <= 16 ? 2LL : 1LL) * sms * THREADS ? 2 : 4);
     if (most_tokens > 1 && spt == 2) {
         if (p.Ns <= 8) return launch_scan<T, 4, 2>(p, n_requests, most_tokens, stream);
         if (p.Ns <= 16) return launch_scan<T, 8, 2>(p, n_requests, most_tokens, stream);
