@@ -1,7 +1,8 @@
 """Rotation of pairs of dims by position ("rotary" encoding), as constants for the kernels that apply it:
 pair i of `dims` dims turns by position * base^(-2 i / dims), optionally stretched for long contexts
-(spec.FrequencyRampSpec: by pair number, spec.FrequencyBandsSpec: by wave length).  The frequencies are computed in 64-bit on the host and rounded once to 32-bit; the angle
-itself (position * frequency) and its sine and cosine are computed in 32-bit inside the kernels."""
+(spec.FrequencyRampSpec: by pair number, spec.FrequencyBandsSpec: by wave length).  The frequencies are computed in
+64-bit on the host and rounded once to 32-bit; the angle itself (position * frequency) and its sine and cosine are
+computed in 32-bit inside the kernels."""
 from __future__ import annotations
 
 import math
