@@ -9,7 +9,7 @@ from .config.generation_config import (BlkSparseAttnConfig, ContinuousBatchingCo
 
 _LAZY = {"OPTForSampling": ".opt.model", "OPTForGreedySearch": ".opt.model", "VononexForSampling": ".vononex.model", "PifelixForSampling": ".pifelix.model",
          "TutelixForSampling": ".tutelix.model", "VoziraxForSampling": ".vozirax.model",
-         "ResatarForSampling": ".resatar.model",
+         "ResatarForSampling": ".resatar.model", "TaboraxForSampling": ".taborax.model",
          "NeuronAutoModelForCausalLM": ".modeling_auto", "HuggingFaceGenerationModelAdapter": ".generation_utils"}
 
 

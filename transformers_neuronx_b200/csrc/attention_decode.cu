@@ -3,6 +3,7 @@
 // value of the live requests is read once per layer and step.
 //
 //   s_j = scale * <q, k_j>  (32-bit; less a distance bias where one is given),  out = sum_j exp(s_j - max) v_j / sum_j exp(s_j - max)
+//   (with a sink, exp(sink - max) more in the denominator: the first warp of the first split starts from it)
 //
 // Grid (heads, rows, splits): a CTA takes one (row, head) and one contiguous range of the pages that hold visible keys
 // (behind a window the pages before it are not counted; those of the first keys that are kept come first); its
@@ -37,6 +38,7 @@ struct DecodeParams {
     float scale;
     int keep_first;                  // with a window: the first positions that stay visible
     DistanceBias bias;
+    SoftmaxSink sink;
     int n_splits, pages_per_split;
     float* scratch;                  // [rows][heads][splits][head_dim + 2]
     int* counters;                   // [rows][heads], zero between calls
@@ -108,7 +110,9 @@ attention_decode_kernel(const DecodeParams p) {
     float m[REP], l[REP], acc[REP][E][8];
 #pragma unroll
     for (int x = 0; x < REP; ++x) {
-        m[x] = -INFINITY; l[x] = 0.f;
+        const bool sink_here = p.sink.on && split == 0 && warp == 0;
+        m[x] = sink_here ? p.sink.score : -INFINITY;
+        l[x] = sink_here && kgrp == 0 ? 1.f : 0.f;             // counted once: the sum runs over the key groups' lanes
 #pragma unroll
         for (int e = 0; e < E; ++e)
 #pragma unroll
@@ -479,7 +483,8 @@ TNX_EXPORT int tnx_attention_decode_append(const void* q, int q_stride, void* ca
                                            int page_size, int window, float scale, int n_splits, int pages_per_split,
                                            float* scratch, int* counters, const void* k_new, const void* v_new,
                                            int kv_stride, int warps, int heads_per_block, int keep_first,
-                                           const float* bias_mul, const float* bias_rate, cudaStream_t stream) {
+                                           const float* bias_mul, const float* bias_rate, int has_sink, float sink_score,
+                                           cudaStream_t stream) {
     // heads_per_block: 1, or what tnx_attention_decode_heads_per_block answers for these sizes (the caller chooses:
     // taking a key/value head's query heads together pays once there are enough (row, key/value head) pairs to fill
     // the GPU; with few rows one block per query head spreads the same work over more blocks).
@@ -494,6 +499,7 @@ TNX_EXPORT int tnx_attention_decode_append(const void* q, int q_stride, void* ca
     if (keep_first < 0 || (bias_mul && !bias_rate)) return TNX_ERR_BAD_ARG;
     DecodeParams p;
     p.keep_first = keep_first; p.bias.mul = bias_mul; p.bias.rate = bias_rate;
+    p.sink.on = has_sink; p.sink.score = sink_score;
     p.q = (const h16*)q; p.q_stride = q_stride; p.cache = (const h16*)cache;
     p.block_tables = block_tables; p.bt_stride = bt_stride; p.rows = rows; p.token_request = token_request;
     p.positions = positions; p.out = (h16*)out; p.out_stride = out_stride;
@@ -536,7 +542,7 @@ TNX_EXPORT int tnx_attention_decode(const void* q, int q_stride, const void* cac
     return tnx_attention_decode_append(q, q_stride, const_cast<void*>(cache), block_tables, bt_stride, rows, token_request,
                                        positions, out, out_stride, n_rows, n_heads, n_kv_heads, head_dim, page_size, window,
                                        scale, n_splits, pages_per_split, scratch, counters, nullptr, nullptr, 0, 4, 1, 0, nullptr,
-                                       nullptr, stream);
+                                       nullptr, 0, 0.f, stream);
 }
 
 // ---------------------------------------------------------------------------------------------------

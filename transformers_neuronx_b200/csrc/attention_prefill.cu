@@ -31,6 +31,7 @@ struct PrefillParams {
     float scale_log2;                // scale * log2(e)
     int keep_first;
     DistanceBias bias;
+    SoftmaxSink sink;
 };
 
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -115,13 +116,17 @@ attention_prefill_kernel(const PrefillParams p) {
 #pragma unroll
     for (int i = 0; i < HEAD / 8; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
     float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+    const float scale_log2 = BIAS ? 1.f : p.scale_log2;      // of the scores as they are carried
+    if (p.sink.on) {                                         // the running maximum in the scores' own units, the sum over a row's four lanes
+        m_run[0] = m_run[1] = p.sink.score * 1.4426950408889634f / scale_log2;
+        l_run[0] = l_run[1] = (lane & 3) == 0 ? 1.f : 0.f;
+    }
     const int r_lo = warp * 16 + (lane >> 2);                // this thread's two rows within the tile
     const int qpos_lo = pos0 + r_lo, qpos_hi = qpos_lo + 8;
 
     // p.window: the mask rule of common.cuh; tiles of keys are numbered along the walk over the visible ones
     const BlockWalk walk = walk_blocks(first_visible_key(pos0, p.window), p.keep_first, BKV);
     const int n_tiles = walk.count(pos_last / BKV);
-    const float scale_log2 = BIAS ? 1.f : p.scale_log2;      // of the scores as they are carried
     float bias_mul = 0.f, bias_rate = 0.f;
     if (BIAS) { bias_mul = p.bias.mul[h]; bias_rate = p.bias.rate[h]; }
     const int first_lo = first_visible_key(qpos_lo, p.window), first_hi = first_visible_key(qpos_hi, p.window);
@@ -306,7 +311,7 @@ TNX_EXPORT int tnx_attention_prefill(const void* q, int q_stride, const void* ca
                                      const int* q_len, const int* ctx_len, void* out, int out_stride, int n_items,
                                      int n_heads, int n_kv_heads, int head_dim, int page_size, int window,
                                      float scale, int keep_first, const float* bias_mul, const float* bias_rate,
-                                     cudaStream_t stream) {
+                                     int has_sink, float sink_score, cudaStream_t stream) {
     if (n_items <= 0) return 0;
     if (page_size != PAGE || head_dim % 16 || head_dim < 16 || head_dim > 256 || n_kv_heads <= 0 ||
         n_heads % n_kv_heads || q_stride % 8 || out_stride % 2 || ((uintptr_t)q & 15) || ((uintptr_t)cache & 15) ||
@@ -315,6 +320,7 @@ TNX_EXPORT int tnx_attention_prefill(const void* q, int q_stride, const void* ca
     if (keep_first < 0 || (bias_mul && !bias_rate)) return TNX_ERR_BAD_ARG;
     PrefillParams p;
     p.keep_first = keep_first; p.bias.mul = bias_mul; p.bias.rate = bias_rate;
+    p.sink.on = has_sink; p.sink.score = sink_score;
     p.q = (const h16*)q; p.q_stride = q_stride; p.cache = (const h16*)cache; p.block_tables = block_tables;
     p.bt_stride = bt_stride; p.tile_req = tile_req; p.tile_q0 = tile_q0; p.q_start = q_start; p.q_len = q_len;
     p.ctx_len = ctx_len; p.out = (h16*)out; p.out_stride = out_stride; p.n_heads = n_heads; p.n_kv_heads = n_kv_heads;

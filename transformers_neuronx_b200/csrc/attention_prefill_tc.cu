@@ -61,6 +61,7 @@ struct TcPrefillParams {
     float scale_log2;
     int keep_first;              // with a window: the first positions that stay visible
     DistanceBias bias;
+    SoftmaxSink sink;
     int* err;
 };
 
@@ -292,6 +293,7 @@ attention_prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __g
         const int qpos = pos0 + r;
         const int first_key = first_visible_key(qpos, p.window);
         float m_run = -INFINITY, l_run = 0.f;
+        if (p.sink.on) { m_run = p.sink.score * 1.4426950408889634f; l_run = 1.f; }
         const float scale_log2 = BIAS ? 1.f : p.scale_log2;      // of the scores as they are carried
         float bias_mul = 0.f, bias_rate = 0.f;
         if constexpr (BIAS) { bias_mul = p.bias.mul[h]; bias_rate = p.bias.rate[h]; }
@@ -447,7 +449,8 @@ TNX_EXPORT int tnx_attention_prefill_tc(const void* q, int q_stride, int n_rows_
                                         const int* q_start, const int* q_len, const int* ctx_len, void* out,
                                         int out_stride, int n_items, int n_heads, int n_kv_heads, int head_dim,
                                         int page_size, int window, float scale, int keep_first, const float* bias_mul,
-                                        const float* bias_rate, int* err_word, cudaStream_t stream) {
+                                        const float* bias_rate, int has_sink, float sink_score, int* err_word,
+                                        cudaStream_t stream) {
     if (n_items <= 0) return 0;
     if (head_dim < 64 || head_dim > 128 || head_dim % 16 || page_size != PAGE || n_kv_heads <= 0 || n_heads % n_kv_heads || q_stride % 8 ||
         out_stride % 8 || ((uintptr_t)q & 15) || ((uintptr_t)cache & 15) || ((uintptr_t)out & 15) ||
@@ -461,6 +464,7 @@ TNX_EXPORT int tnx_attention_prefill_tc(const void* q, int q_stride, int n_rows_
     p.block_tables = block_tables; p.bt_stride = bt_stride; p.tile_req = tile_req; p.tile_q0 = tile_q0;
     p.q_start = q_start; p.q_len = q_len; p.ctx_len = ctx_len; p.out = (h16*)out; p.out_stride = out_stride;
     p.n_heads = n_heads; p.n_kv_heads = n_kv_heads; p.window = window; p.scale_log2 = scale * 1.4426950408889634f;
+    p.sink.on = has_sink; p.sink.score = sink_score;
     p.err = err_word; p.keep_first = keep_first; p.bias.mul = bias_mul; p.bias.rate = bias_rate;
     switch (head_dim) {
         case 128: return launch_tc<128, 2, 3>(mq, mkv, p, n_heads, n_items, stream);

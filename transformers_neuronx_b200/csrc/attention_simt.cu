@@ -21,7 +21,8 @@ attention_simt_kernel(const T* __restrict__ q, int q_stride, const T* __restrict
                       const int* __restrict__ block_tables, int bt_stride,
                       const int* __restrict__ token_request, const int* __restrict__ positions,
                       T* __restrict__ out, int out_stride, int n_tokens, int n_heads, int n_kv_heads,
-                      int head_dim, int page_size, int window, float scale, int keep_first, DistanceBias bias) {
+                      int head_dim, int page_size, int window, float scale, int keep_first, DistanceBias bias,
+                      SoftmaxSink sink) {
     extern __shared__ float qsm[];                  // [warps per block][head_dim]
     pdl_launch_dependents();
     pdl_wait();
@@ -40,7 +41,7 @@ attention_simt_kernel(const T* __restrict__ q, int q_stride, const T* __restrict
     __syncwarp();
 
     const size_t head_block = (size_t)page_size * head_dim;
-    float m = -INFINITY, l = 0.f;
+    float m = sink.on ? sink.score : -INFINITY, l = sink.on ? 1.f : 0.f;
     float acc[MAX_DIMS_PER_LANE];
 #pragma unroll
     for (int i = 0; i < MAX_DIMS_PER_LANE; ++i) acc[i] = 0.f;
@@ -97,12 +98,13 @@ TNX_EXPORT int tnx_attention_simt(const void* q, int q_stride, const void* cache
                                   int bt_stride, const int* token_request, const int* positions, void* out,
                                   int out_stride, int n_tokens, int n_heads, int n_kv_heads, int head_dim,
                                   int page_size, int window, float scale, int keep_first, const float* bias_mul,
-                                  const float* bias_rate, int is_h16, cudaStream_t stream) {
+                                  const float* bias_rate, int has_sink, float sink_score, int is_h16, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (head_dim <= 0 || head_dim > 32 * WIDE_DIMS_PER_LANE || n_kv_heads <= 0 || n_heads % n_kv_heads)
         return TNX_ERR_UNSUPPORTED;
     if (keep_first < 0 || (bias_mul && !bias_rate)) return TNX_ERR_BAD_ARG;
     const DistanceBias bias{bias_mul, bias_rate};
+    const SoftmaxSink sink{has_sink, sink_score};
     const int warps = 4;
     const long long pairs = (long long)n_tokens * n_heads;
     const int blocks = (int)((pairs + warps - 1) / warps);
@@ -111,7 +113,7 @@ TNX_EXPORT int tnx_attention_simt(const void* q, int q_stride, const void* cache
     return tnx_launch_in_order(attention_simt_kernel<T, DPL>, dim3(blocks), dim3(warps * 32), smem, stream, (const T*)q,\
                                q_stride, (const T*)cache, block_tables, bt_stride, token_request, positions, (T*)out,   \
                                out_stride, n_tokens, n_heads, n_kv_heads, head_dim, page_size, window, scale, keep_first,   \
-                               bias)
+                               bias, sink)
     if (head_dim <= 256) {
         if (is_h16) ASIMT(h16, 8);
         ASIMT(float, 8);

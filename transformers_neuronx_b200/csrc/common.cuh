@@ -108,7 +108,7 @@ template <> __device__ __forceinline__ h16 from_float<h16>(float v) { return flo
 
 // Activations that a product's epilogue applies to (sum + bias), by code: the names of
 // src/transformers_neuronx/activations.py (relu :43-48, gelu_new :17-41 with its tanh form, sigmoid
-// :66-67, silu :70-72) plus the exact (erf) gelu.  The code travels to the kernel as a number, so
+// :66-67, silu :70-72) plus the exact (erf) gelu and the square of relu.  The code travels to the kernel as a number, so
 // another activation is one more case here and one more name in kernels/ops.py.
 #define TNX_ACT_NONE 0
 #define TNX_ACT_RELU 1
@@ -116,8 +116,9 @@ template <> __device__ __forceinline__ h16 from_float<h16>(float v) { return flo
 #define TNX_ACT_SILU 3
 #define TNX_ACT_SIGMOID 4
 #define TNX_ACT_GELU 5
-#define TNX_ACT_COUNT 6
-// The two cheap cases are inline; everything else is one call into a function that is compiled once.
+#define TNX_ACT_RELU2 6
+#define TNX_ACT_COUNT 7
+// The cheap cases are inline; everything else is one call into a function that is compiled once.
 // (With every case expanded inline, the epilogues of the tensor-core products, which apply the
 // activation to several accumulators per loop turn, grew so much that a 2,048-token prefill of the
 // 6.7B sizes took 32 ms instead of 26: also for the products that use no activation at all.)
@@ -170,6 +171,7 @@ template <> struct Vec8<float> {
 __device__ __forceinline__ float apply_activation(float v, int act) {
     if (act == TNX_ACT_NONE) return v;
     if (act == TNX_ACT_RELU) return fmaxf(v, 0.f);
+    if (act == TNX_ACT_RELU2) { const float r = fmaxf(v, 0.f); return r * r; }
     return apply_activation_other(v, act);
 }
 
@@ -205,6 +207,13 @@ __host__ __device__ __forceinline__ BlockWalk walk_blocks(int first_key, int kee
 struct DistanceBias {
     const float* mul;
     const float* rate;
+};
+// One more key for every query and head, of a fixed score and without a value: the softmax's denominator gains exp(score).
+// A kernel starts its running (maximum, sum) at (score, 1) instead of (-inf, 0); kernels that split a row's keys do so in
+// one of the parts.
+struct SoftmaxSink {
+    int on;
+    float score;
 };
 __device__ __forceinline__ float log2_approx(float x) {
     float y;

@@ -7,9 +7,13 @@
 //                         y = g * sigmoid(alpha g) * (u + up_shift),  result W_down y
 //   out = sum_j expert_{e_j}(w_j h)   (weight on the input)    or    sum_j w_j expert_{e_j}(h)   (on the output)
 //   an expert without a gate (form 1):  y = relu(W_up x)^2,  result W_down y
-//   routing options (sigmoid scores): a correction per expert added to the scores for the CHOICE only; experts in equal
+//   routing options: a correction per expert added to the scores for the CHOICE only; experts in equal
 //   groups of neighbours, a group scored by the sum of its group_top largest choice scores, only the keep_groups best
 //   groups' experts open to the choice; weights w_j / (sum_j w_j + renorm_eps) * weight_scale
+//   identity experts: the last n_identity of the router's outputs return their input, w_j h, and have no matrices; in the
+//   lists of choices they stand as IDENTITY
+//   a gate: one more row of the router's matrix, sigmoid(W_gate h) per token, is the weight of the experts that every
+//   token takes (or is written out, for a shared feed-forward that runs on its own)
 //
 // Kernels of this file (T: the activations' type, TW: the stored type of the experts' matrices):
 //   moe_router_kernel      a block a token: logits, scores, the top experts and their weights
@@ -25,6 +29,7 @@
 namespace {
 constexpr int MAX_TOP = 16;
 constexpr int MAX_EXPERTS = 1024;
+constexpr int IDENTITY = -2;      // in a list of choices: the token itself (-1: a padded row, no expert)
 
 // 8 elements of a matrix as they are loaded (converted when they are used, so that several loads can be in flight).
 template <typename TW> struct Raw8;
@@ -79,7 +84,11 @@ struct RouterOptions {
     int n_groups, keep_groups, group_top;
     float renorm_eps, weight_scale;
     const float* bias;           // [E], added to the logits, or null
-    int always;                  // further experts (E, E + 1, ...) that every token takes with weight 1, behind the chosen ones
+    int always;                  // further experts that every token takes, behind the chosen ones: numbers E - n_identity on,
+                                 // weight 1, or the gate
+    int n_identity;              // the last n_identity of the E outputs are identity experts
+    int gated;                   // row E of the router's matrix gives the gate
+    float* gate_out;             // [N]: where the gate goes, or null
 };
 
 template <typename T, typename TW>
@@ -87,10 +96,10 @@ __global__ void __launch_bounds__(128)
 moe_router_kernel(const T* __restrict__ h, int ld, const TW* __restrict__ wr, const int* __restrict__ token_request,
                   int* __restrict__ ids, float* __restrict__ weights, int W, int E, int top, int softmax_scores,
                   int renormalize, RouterOptions ro) {
-    extern __shared__ __align__(16) float sm[];            // [W] the row, [E] the logits (or choice scores), [E] the scores, [E] groups
+    extern __shared__ __align__(16) float sm[];            // [W] the row, [E + 1] the logits (or choice scores; the gate's), [E] the scores, [E] groups
     float* x = sm;
     float* z = sm + ((W + 3) & ~3);
-    float* sc = z + E;
+    float* sc = z + E + 1;
     float* gscore = sc + E;
     pdl_launch_dependents();
     pdl_wait();
@@ -98,24 +107,32 @@ moe_router_kernel(const T* __restrict__ h, int ld, const TW* __restrict__ wr, co
     const size_t row = (size_t)n * (top + ro.always);        // where the token's experts and weights begin
     if (token_request[n] < 0) {                              // a padded row of a captured step: no expert
         if (threadIdx.x < top + ro.always) { ids[row + threadIdx.x] = -1; weights[row + threadIdx.x] = 0.f; }
+        if (threadIdx.x == 0 && ro.gate_out) ro.gate_out[n] = 0.f;
         return;
     }
     for (int c = threadIdx.x; c < W; c += blockDim.x) x[c] = to_float(h[(size_t)n * ld + c]);
     __syncthreads();
     const bool vec = W % 8 == 0 && ((uintptr_t)wr % 16) == 0;
-    for (int e = warp; e < E; e += 4) {
+    for (int e = warp; e < E + ro.gated; e += 4) {
         const float s = warp_dot<TW>(wr + (size_t)e * W, x, W, lane, vec);
-        if (lane == 0) z[e] = s + (ro.bias ? ro.bias[e] : 0.f);
+        if (lane == 0) z[e] = s + (ro.bias && e < E ? ro.bias[e] : 0.f);
     }
     __syncthreads();
     if (warp != 0) return;
     // The choice is made on the logits: both scores grow with them, and a sigmoid that has run out of bits near 1
     // would tie experts that their logits still tell apart.  With a correction or groups the choice is made on
-    // choice score = sigmoid + correction, as the design says, and the weight is the uncorrected sigmoid.
+    // choice score = score + correction, as the designs say, and the weight is the uncorrected score.
     const bool corrected = ro.correction != nullptr || ro.n_groups > 1;
+    float mx = -INFINITY, sum = 0.f;
+    if (softmax_scores) {
+        for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
+        mx = warp_max(mx);
+        for (int e = lane; e < E; e += 32) sum += expf(z[e] - mx);
+        sum = warp_sum(sum);
+    }
     if (corrected) {
         for (int e = lane; e < E; e += 32) {
-            const float s0 = 1.f / (1.f + expf(-z[e]));
+            const float s0 = softmax_scores ? expf(z[e] - mx) / sum : 1.f / (1.f + expf(-z[e]));
             sc[e] = s0;
             z[e] = s0 + (ro.correction ? ro.correction[e] : 0.f);
         }
@@ -161,13 +178,6 @@ moe_router_kernel(const T* __restrict__ h, int ld, const TW* __restrict__ wr, co
             __syncwarp();
         }
     }
-    float mx = -INFINITY, sum = 0.f;
-    if (softmax_scores) {
-        for (int e = lane; e < E; e += 32) mx = fmaxf(mx, z[e]);
-        mx = warp_max(mx);
-        for (int e = lane; e < E; e += 32) sum += expf(z[e] - mx);
-        sum = warp_sum(sum);
-    }
     float chosen_w[MAX_TOP];
     int chosen[MAX_TOP];
     float total = 0.f;
@@ -184,7 +194,8 @@ moe_router_kernel(const T* __restrict__ h, int ld, const TW* __restrict__ wr, co
             const int oa = __shfl_xor_sync(0xffffffffu, arg, o);
             if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
         }
-        chosen[j] = arg;
+        if (arg >= E) arg = 0;                              // every score left is NaN: any expert gives NaN
+        chosen[j] = arg >= E - ro.n_identity ? IDENTITY : arg;
         chosen_w[j] = corrected ? sc[arg] : (softmax_scores ? expf(best - mx) / sum : 1.f / (1.f + expf(-best)));
         total += chosen_w[j];
         if (lane == 0) z[arg] = -INFINITY;
@@ -195,7 +206,9 @@ moe_router_kernel(const T* __restrict__ h, int ld, const TW* __restrict__ wr, co
             ids[row + j] = chosen[j];
             weights[row + j] = (renormalize ? chosen_w[j] / (total + ro.renorm_eps) : chosen_w[j]) * ro.weight_scale;
         }
-        for (int j = 0; j < ro.always; ++j) { ids[row + top + j] = E + j; weights[row + top + j] = 1.f; }
+        const float gate = ro.gated ? 1.f / (1.f + expf(-z[E])) : 1.f;
+        for (int j = 0; j < ro.always; ++j) { ids[row + top + j] = E - ro.n_identity + j; weights[row + top + j] = gate; }
+        if (ro.gate_out) ro.gate_out[n] = gate;
     }
 }
 
@@ -413,19 +426,22 @@ moe_down_kernel(const T* __restrict__ y, const TW* __restrict__ down, const int*
 }
 
 // out[n] (+)= sum over the token's choices, in their order, of per_pair (times the choice's weight where it multiplies
-// the expert's output).
+// the expert's output; an identity expert's is weight * h[n]).
+template <typename T>
 __global__ void __launch_bounds__(128)
-moe_sum_kernel(const float* __restrict__ per_pair, const int* __restrict__ ids, const float* __restrict__ weights, float* out,
-               int W, int top, int accumulate, int weight_on_input) {
+moe_sum_kernel(const float* __restrict__ per_pair, const T* __restrict__ h, int ld, const int* __restrict__ ids,
+               const float* __restrict__ weights, float* out, int W, int top, int accumulate, int weight_on_input) {
     pdl_launch_dependents();
     pdl_wait();
     const int n = blockIdx.x;
-    if (ids[(size_t)n * top] < 0) return;                   // a padded row of a captured step
+    if (ids[(size_t)n * top] == -1) return;                 // a padded row of a captured step
     for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < W; c += gridDim.y * blockDim.x) {
         float s = 0.f;
         for (int j = 0; j < top; ++j) {
-            const float v = per_pair[((size_t)n * top + j) * W + c];
-            s += weight_on_input ? v : v * weights[(size_t)n * top + j];
+            const size_t pair = (size_t)n * top + j;
+            const bool self = ids[pair] == IDENTITY;
+            const float v = self ? to_float(h[(size_t)n * ld + c]) : per_pair[pair * W + c];
+            s += weight_on_input && !self ? v : v * weights[pair];
         }
         float* dst = out + (size_t)n * W + c;
         *dst = accumulate ? *dst + s : s;
@@ -436,16 +452,19 @@ moe_sum_kernel(const float* __restrict__ per_pair, const int* __restrict__ ids, 
 TNX_EXPORT int tnx_moe_route(const void* h, int ld, const void* router, const int* token_request, int* ids, float* weights,
                              int N, int W, int E, int top, int softmax_scores, int renormalize, int h_h16, int w_h16,
                              const float* correction, int n_groups, int keep_groups, int group_top, float renorm_eps,
-                             float weight_scale, const float* bias, int always, cudaStream_t stream) {
+                             float weight_scale, const float* bias, int always, int n_identity, int gated, float* gate_out,
+                             cudaStream_t stream) {
+    // E: the router's outputs, identity experts included; `router` has E rows, with `gated` one more
     if (N <= 0) return 0;
     if (W <= 0 || E <= 0 || E > MAX_EXPERTS || top <= 0 || top > MAX_TOP || top > E) return TNX_ERR_UNSUPPORTED;
     if (always < 0 || top + always > MAX_TOP || E + always > MAX_EXPERTS) return TNX_ERR_UNSUPPORTED;
+    if (n_identity < 0 || n_identity >= E || gated < 0 || gated > 1 || (gate_out && !gated)) return TNX_ERR_BAD_ARG;
     if (n_groups < 1 || E % n_groups || keep_groups < 1 || keep_groups > n_groups || group_top < 1 ||
-        (long long)keep_groups * (E / n_groups) < top || ((correction || n_groups > 1) && softmax_scores))
+        (long long)keep_groups * (E / n_groups) < top)
         return TNX_ERR_BAD_ARG;
     if (n_groups > 1 && E / n_groups > 64 && group_top > 1) return TNX_ERR_UNSUPPORTED;
-    const RouterOptions ro{correction, n_groups, keep_groups, group_top, renorm_eps, weight_scale, bias, always};
-    const size_t smem = (size_t)(((W + 3) & ~3) + 3 * E) * sizeof(float);
+    const RouterOptions ro{correction, n_groups, keep_groups, group_top, renorm_eps, weight_scale, bias, always, n_identity, gated, gate_out};
+    const size_t smem = (size_t)(((W + 3) & ~3) + 3 * E + 1) * sizeof(float);
     if (smem > 160 * 1024) return TNX_ERR_UNSUPPORTED;
 #define GO(T, TW)                                                                                                       \
     do {                                                                                                                \
@@ -488,8 +507,9 @@ TNX_EXPORT int tnx_moe_experts(const void* h, int ld, const void* gate_up, const
         rc = tnx_launch_in_order(moe_down_kernel<T, TW>, g2, dim3(128), smem2, stream, (const T*)y, (const TW*)down,    \
                                  ids, per_pair, W, F, pairs, per2);                                                     \
         if (rc != 0) return rc;                                                                                         \
-        return tnx_launch_in_order(moe_sum_kernel, dim3(N, N >= 256 ? 1 : (W + 511) / 512), dim3(128), 0, stream, (const float*)per_pair, ids, weights, \
-                                   out, W, top, accumulate, weight_on_input);                                           \
+        return tnx_launch_in_order(moe_sum_kernel<T>, dim3(N, N >= 256 ? 1 : (W + 511) / 512), dim3(128), 0, stream,    \
+                                   (const float*)per_pair, (const T*)h, ld, ids, weights, out, W, top, accumulate,      \
+                                   weight_on_input);                                                                    \
     } while (0)
     if (h_h16 && w_h16) GO(h16, h16);
     if (h_h16) GO(h16, float);

@@ -10,6 +10,7 @@
 //   moe_act_kernel       y = g * sigmoid(alpha g) * (u + up_shift), g and u clamped, from the gate/up product's output
 //                        (moe_act_relu2_kernel: y = relu(u)^2 for experts without a gate)
 //   moe_combine_kernel   out[token] (+)= sum over the token's pairs, in the order of the choice, of the down product's rows
+//                        (a pair whose expert is the token itself takes no row: weight * h[token])
 //
 // Nothing is read on the host: the sizes of the buffers follow from the numbers of tokens and experts alone (at most
 // pairs / tile + experts tiles), so a step can be captured in a CUDA graph.
@@ -17,6 +18,7 @@
 
 namespace {
 constexpr int MAX_EXPERTS = 1024;
+constexpr int IDENTITY = -2;      // of a pair's expert, and then of its row: the token itself (-1: a padded row)
 
 __global__ void __launch_bounds__(1024)
 moe_plan_kernel(const int* __restrict__ ids, int n_pairs, int n_experts, int max_tiles, int TILE, int* __restrict__ group_of_tile,
@@ -44,7 +46,7 @@ moe_plan_kernel(const int* __restrict__ ids, int n_pairs, int n_experts, int max
     __syncthreads();
     for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) {
         const int e = ids[i];
-        row_of_pair[i] = e >= 0 ? first[e] + atomicAdd(&cursor[e], 1) : -1;
+        row_of_pair[i] = e >= 0 ? first[e] + atomicAdd(&cursor[e], 1) : e;
     }
 }
 
@@ -124,17 +126,19 @@ moe_act_relu2_kernel(const h16* __restrict__ u, h16* __restrict__ y, const int* 
 }
 
 __global__ void __launch_bounds__(128)
-moe_combine_kernel(const float* __restrict__ rows, const int* __restrict__ row_of_pair, const float* __restrict__ weights,
-                   float* out, int W, int top, int accumulate, int weight_on_input) {
+moe_combine_kernel(const float* __restrict__ rows, const h16* __restrict__ h, int ld, const int* __restrict__ row_of_pair,
+                   const float* __restrict__ weights, float* out, int W, int top, int accumulate, int weight_on_input) {
     pdl_launch_dependents();
     pdl_wait();
     const int n = blockIdx.x;
-    if (row_of_pair[(size_t)n * top] < 0) return;                 // a padded row of a captured step
+    if (row_of_pair[(size_t)n * top] == -1) return;               // a padded row of a captured step
     for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < W; c += gridDim.y * blockDim.x) {
         float s = 0.f;
         for (int j = 0; j < top; ++j) {
-            const float v = rows[(size_t)row_of_pair[(size_t)n * top + j] * W + c];
-            s += weight_on_input ? v : v * weights[(size_t)n * top + j];
+            const int row = row_of_pair[(size_t)n * top + j];
+            const bool self = row == IDENTITY;
+            const float v = self ? h16_to_float(h[(size_t)n * ld + c]) : rows[(size_t)row * W + c];
+            s += weight_on_input && !self ? v : v * weights[(size_t)n * top + j];
         }
         float* dst = out + (size_t)n * W + c;
         *dst = accumulate ? *dst + s : s;
@@ -173,10 +177,10 @@ TNX_EXPORT int tnx_moe_act(const void* gu, void* y, const int* group_of_tile, in
                                group_of_tile, tile, F, gate_max, up_min, up_max, alpha, up_shift);
 }
 
-TNX_EXPORT int tnx_moe_combine(const float* rows, const int* row_of_pair, const float* weights, float* out, int N, int W, int top,
+TNX_EXPORT int tnx_moe_combine(const float* rows, const void* h, int ld, const int* row_of_pair, const float* weights, float* out, int N, int W, int top,
                                int accumulate, int weight_on_input, cudaStream_t stream) {
     if (N <= 0) return 0;
     // few tokens: a slice of the width a block, so that the loads of a row are asked for together
-    return tnx_launch_in_order(moe_combine_kernel, dim3(N, N >= 256 ? 1 : (W + 511) / 512), dim3(128), 0, stream, rows, row_of_pair, weights, out, W, top,
+    return tnx_launch_in_order(moe_combine_kernel, dim3(N, N >= 256 ? 1 : (W + 511) / 512), dim3(128), 0, stream, rows, (const h16*)h, ld, row_of_pair, weights, out, W, top,
                                accumulate, weight_on_input);
 }

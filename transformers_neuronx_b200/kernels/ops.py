@@ -91,7 +91,7 @@ _FLOATS = (torch.float32,) + _H16
 # Activations a product's epilogue applies, by the names the reference looks up
 # (src/transformers_neuronx/hlo.py:485-501 -> activations.py) -> the kernels' codes (csrc/common.cuh).
 ACTIVATIONS = {None: 0, "none": 0, "relu": 1, "gelu_new": 2, "gelu_new_legacy": 2, "gelu_pytorch_tanh": 2,
-               "silu": 3, "swish": 3, "sigmoid": 4, "gelu": 5}
+               "silu": 3, "swish": 3, "sigmoid": 4, "gelu": 5, "relu2": 6}
 
 
 def activation_code(name) -> int:
@@ -280,19 +280,20 @@ def mask_rule(window=0, chunk=0) -> int:
     return -chunk if chunk else window
 
 
-def _kept_and_bias(keep_first, bias, n_heads, window):
-    """The attention kernels' last arguments: how many first positions stay visible beside a window, and the distance
-    bias (mul, rate), 32-bit [n_heads] each: mul[h] * ln(1 + rate[h] * (i - j)) is taken off the scores (None: none)."""
+def _score_options(keep_first, bias, sink, n_heads, window):
+    """The attention kernels' last arguments: how many first positions stay visible beside a window; the distance
+    bias (mul, rate), 32-bit [n_heads] each: mul[h] * ln(1 + rate[h] * (i - j)) is taken off the scores (None: none); the
+    sink, a number: every softmax has exp(sink) more in its denominator (None: none)."""
     keep_first = int(keep_first or 0)
     if keep_first < 0 or (keep_first and not window):
         raise KernelError("keep_first is a number of positions kept beside a window")
     mul, rate = bias if bias is not None else (None, None)
     _f32_vec(mul, "the bias's multiplier", n_heads); _f32_vec(rate, "the bias's rate", n_heads)
-    return c_int(keep_first), _p(mul), _p(rate)
+    return c_int(keep_first), _p(mul), _p(rate), c_int(0 if sink is None else 1), c_float(0.0 if sink is None else float(sink))
 
 
 def attention_simt(q, cache, block_tables, token_request, positions, out, n_heads, scale, window=0, chunk=0, keep_first=0,
-                   bias=None):
+                   bias=None, sink=None):
     """q: [N, n_heads * head_dim] view; out likewise; cache as in kv_append."""
     lib = _lib("attention_simt", cache, q, out)
     _need(cache, "cache", _FLOATS, 5)
@@ -307,7 +308,7 @@ def attention_simt(q, cache, block_tables, token_request, positions, out, n_head
     _check(lib.tnx_attention_simt(_p(q), c_int(q_stride), _p(cache), _p(block_tables), c_int(block_tables.stride(0)),
                                   _p(token_request), _p(positions), _p(out), c_int(out_stride), c_int(N),
                                   c_int(n_heads), c_int(n_kv), c_int(d), c_int(ps), c_int(mask_rule(window, chunk)),
-                                  c_float(scale), *_kept_and_bias(keep_first, bias, n_heads, window),
+                                  c_float(scale), *_score_options(keep_first, bias, sink, n_heads, window),
                                   c_int(_is_h16(cache)), _stream()), "attention_simt")
 
 
@@ -637,7 +638,7 @@ def decode_attention_plan(pairs: int, sms: int, head_dim: int, max_pages: int):
 
 
 def attention_decode(q, cache, block_tables, token_request, positions, out, n_heads, scale, window=0, rows=None,
-                     n_rows=None, max_kv_len=None, n_splits=None, new_kv=None, warps=None, grouped=None, chunk=0, keep_first=0, bias=None):
+                     n_rows=None, max_kv_len=None, n_splits=None, new_kv=None, warps=None, grouped=None, chunk=0, keep_first=0, bias=None, sink=None):
     """One query token per row over the paged 16-bit cache.  `rows` (int32) names the rows of q
     that are decode tokens (None: all); max_kv_len bounds their contexts (for the split plan).
     new_kv = (k, v), [rows of q, kv_heads * head_dim] bfloat16: the keys and values of the rows' own
@@ -718,14 +719,14 @@ def attention_decode(q, cache, block_tables, token_request, positions, out, n_he
         _p(rows), _p(token_request), _p(positions), _p(out), c_int(out_stride), c_int(R),
         c_int(n_heads), c_int(n_kv), c_int(d), c_int(ps), c_int(mask_rule(window, chunk)), c_float(scale),
         c_int(n_splits), c_int(pps), _p(scratch), _p(st.get("att_counters")), _p(k_new), _p(v_new), c_int(kv_stride),
-        c_int(warps), c_int(heads_per_block), *_kept_and_bias(keep_first, bias, n_heads, window), _stream()), "attention_decode")
+        c_int(warps), c_int(heads_per_block), *_score_options(keep_first, bias, sink, n_heads, window), _stream()), "attention_decode")
 
 
 ATTN_PREFILL_TILE = 128      # query rows of one work item of the prefill attention kernel
 
 
 def attention_prefill(q, cache, block_tables, tile_req, tile_q0, q_start, q_len, ctx_len, out, n_heads, scale,
-                      window=0, n_items=None, chunk=0, keep_first=0, bias=None):
+                      window=0, n_items=None, chunk=0, keep_first=0, bias=None, sink=None):
     """Causal attention of prompt portions: work items (request, first row of an ATTN_PREFILL_TILE-row tile)."""
     lib = _lib("attention_prefill", cache, q, out)
     _need(cache, "cache", _H16, 5)
@@ -742,7 +743,7 @@ def attention_prefill(q, cache, block_tables, tile_req, tile_q0, q_start, q_len,
                                      _p(tile_req), _p(tile_q0), _p(q_start), _p(q_len), _p(ctx_len), _p(out),
                                      c_int(out_stride), c_int(n), c_int(n_heads), c_int(n_kv), c_int(d), c_int(ps),
                                      c_int(mask_rule(window, chunk)), c_float(scale),
-                                     *_kept_and_bias(keep_first, bias, n_heads, window), _stream()), "attention_prefill")
+                                     *_score_options(keep_first, bias, sink, n_heads, window), _stream()), "attention_prefill")
 
 
 def attention_prefill_tc_supported(q, cache, out) -> bool:
@@ -753,7 +754,7 @@ def attention_prefill_tc_supported(q, cache, out) -> bool:
 
 
 def attention_prefill_tc(q, cache, block_tables, tile_req, tile_q0, q_start, q_len, ctx_len, out, n_heads, scale,
-                         window=0, n_items=None, chunk=0, keep_first=0, bias=None):
+                         window=0, n_items=None, chunk=0, keep_first=0, bias=None, sink=None):
     """attention_prefill on the tcgen05 tensor cores (head sizes 64 to 128 in steps of 16).  The cache must hold finite
     numbers in every row, written or not (CacheStorage allocates it zeroed)."""
     lib = _lib("attention_prefill_tc", cache, q, out)
@@ -772,11 +773,11 @@ def attention_prefill_tc(q, cache, block_tables, tile_req, tile_q0, q_start, q_l
                                         _p(block_tables), c_int(block_tables.stride(0)), _p(tile_req), _p(tile_q0),
                                         _p(q_start), _p(q_len), _p(ctx_len), _p(out), c_int(out_stride), c_int(n),
                                         c_int(n_heads), c_int(n_kv), c_int(d), c_int(ps), c_int(mask_rule(window, chunk)),
-                                        c_float(scale), *_kept_and_bias(keep_first, bias, n_heads, window), _p(st["err"]),
+                                        c_float(scale), *_score_options(keep_first, bias, sink, n_heads, window), _p(st["err"]),
                                         _stream()), "attention_prefill_tc")
 
 
-def _attention_h16(ctx, group, q, cache, out, n_heads, scale, window, new_kv, chunk=0, keep_first=0, bias=None):
+def _attention_h16(ctx, group, q, cache, out, n_heads, scale, window, new_kv, chunk=0, keep_first=0, bias=None, sink=None):
     if cache.shape[3] != 16 or cache.shape[4] > 256 or q.stride(0) % 8 or q.data_ptr() % 16:
         return False                             # rows wider than 256 dims: the CUDA-core kernel takes up to 768
     bt = ctx.block_tables[group]
@@ -791,33 +792,33 @@ def _attention_h16(ctx, group, q, cache, out, n_heads, scale, window, new_kv, ch
     if ctx.n_prefill_tiles:
         prefill = attention_prefill_tc if attention_prefill_tc_supported(q, cache, out) else attention_prefill
         prefill(q, cache, bt, ctx.tile_req, ctx.tile_q0, ctx.q_start, ctx.q_len, ctx.ctx_len, out,
-                n_heads, scale, window, n_items=ctx.n_prefill_tiles, chunk=chunk, keep_first=keep_first, bias=bias)
+                n_heads, scale, window, n_items=ctx.n_prefill_tiles, chunk=chunk, keep_first=keep_first, bias=bias, sink=sink)
     if ctx.n_decode_rows:
         attention_decode(q, cache, bt, ctx.token_request, ctx.positions, out, n_heads, scale, window,
                          rows=None if ctx.decode_only else ctx.decode_rows, n_rows=ctx.n_decode_rows,
-                         max_kv_len=ctx.max_decode_ctx, new_kv=fused, chunk=chunk, keep_first=keep_first, bias=bias)
+                         max_kv_len=ctx.max_decode_ctx, new_kv=fused, chunk=chunk, keep_first=keep_first, bias=bias, sink=sink)
     return True
 
 
 _attention_impls["h16"] = _attention_h16
 
 
-def attention(ctx, group, q, cache, out, n_heads, scale, window=0, new_kv=None, chunk=0, keep_first=0, bias=None):
+def attention(ctx, group, q, cache, out, n_heads, scale, window=0, new_kv=None, chunk=0, keep_first=0, bias=None, sink=None):
     """Attention of this step's queries over the cache of the running schedule entry.  32-bit
     caches, and head sizes or windows that the 16-bit kernels do not take, run on the CUDA-core
     kernel; a 16-bit cache runs the prefill kernel for requests with several rows and the split
     decode kernel for requests with one.  new_kv = (k, v, slot_mapping): the keys and values of
     this step's tokens, not yet in the cache; they are appended here, by kv_append or (a step of
     decode tokens only, 16-bit) by the decode kernel itself; None: the cache holds them already (a mixer that
-    reads another mixer's pages).  window / chunk: see mask_rule; keep_first, bias: see
-    _kept_and_bias."""
+    reads another mixer's pages).  window / chunk: see mask_rule; keep_first, bias, sink: see
+    _score_options."""
     impl = _attention_impls.get("h16") if cache.dtype in _H16 else None
-    if impl is not None and impl(ctx, group, q, cache, out, n_heads, scale, window, new_kv, chunk, keep_first, bias):
+    if impl is not None and impl(ctx, group, q, cache, out, n_heads, scale, window, new_kv, chunk, keep_first, bias, sink):
         return
     if new_kv is not None:
         kv_append(new_kv[0], new_kv[1], new_kv[2], cache, ctx.page_size)
     attention_simt(q, cache, ctx.block_tables[group], ctx.token_request, ctx.positions, out, n_heads, scale,
-                   window, chunk, keep_first, bias)
+                   window, chunk, keep_first, bias, sink)
 
 
 # ---------------------------------------------------------------------------------------------
@@ -975,33 +976,37 @@ def conv_qkv_prep(proj, col0, conv_w, taps, state, ctx, q_norm, k_norm, eps, inv
 
 def moe_route(h, router, token_request, ids, weights, top, softmax_scores=False, renormalize=False, correction=None,
               n_groups=1, keep_groups=1, group_top=2, renorm_eps=0.0, weight_scale=1.0, bias=None,
-              always=0):
+              always=0, n_identity=0, gated=False, gate_out=None):
     """For every row of h [N, W]: the `top` experts with the largest scores (sigmoid, or softmax, of the 32-bit product
     with router [E, W], plus bias [E] where it is given) into ids [N, top] (int32; -1 for a padded row) and their scores into weights [N, top].
-    correction (32-bit [E]): added to the sigmoid scores for the choice only.  n_groups > 1: the experts form equal groups
+    correction (32-bit [E]): added to the scores for the choice only.  n_groups > 1: the experts form equal groups
     of neighbours, a group's score is the sum of its group_top largest choice scores, and only experts of the keep_groups
     best groups can be chosen.  The weights are divided by (their sum + renorm_eps) with `renormalize`, then multiplied
-    by weight_scale.  always: as many further experts (E, E + 1, ...), with weight 1 each, stand behind the chosen ones in
-    every row (ids and weights are then [N, top + always])."""
+    by weight_scale.  n_identity: the last of the E experts that return their input; they stand as -2 in ids.  always: as
+    many further experts (E - n_identity, ...), with weight 1 each, stand behind the chosen ones in
+    every row (ids and weights are then [N, top + always]).  gated: the router has one row more, whose product's sigmoid is
+    the weight of those instead of 1, and goes into gate_out (32-bit [N]) where that is given."""
     lib = _lib("moe", h, router)
     _need(h, "h", _FLOATS, None, contiguous=False)
     N, W, ld = _rows_2d(h, "h")
     _need(router, "router", _FLOATS, 2)
-    E = router.shape[0]
+    E = router.shape[0] - (1 if gated else 0)
     if router.shape[1] != W:
         raise KernelError("the router's rows must be as long as h's")
     _need(token_request, "token_request", torch.int32, 1)
     _need(ids, "ids", torch.int32, 2); _need(weights, "weights", torch.float32, 2)
     if tuple(ids.shape) != (N, top + always) or tuple(weights.shape) != (N, top + always):
         raise KernelError(f"ids and weights must be [{N}, {top + always}]")
-    _f32_vec(correction, "correction", E); _f32_vec(bias, "bias", E)
+    _f32_vec(correction, "correction", E); _f32_vec(bias, "bias", E); _f32_vec(gate_out, "gate_out", N)
     _check(lib.tnx_moe_route(_p(h), c_int(ld), _p(router), _p(token_request), _p(ids), _p(weights), c_int(N), c_int(W),
                              c_int(E), c_int(top), c_int(1 if softmax_scores else 0), c_int(1 if renormalize else 0),
                              c_int(_is_h16(h)), c_int(_is_h16(router)), _p(correction), c_int(n_groups), c_int(keep_groups),
-                             c_int(group_top), c_float(renorm_eps), c_float(weight_scale), _p(bias), c_int(always), _stream()), "moe_route")
+                             c_int(group_top), c_float(renorm_eps), c_float(weight_scale), _p(bias), c_int(always), c_int(n_identity),
+                             c_int(1 if gated else 0), _p(gate_out), _stream()), "moe_route")
 
 
 EXPERT_FORMS = {"gated_swish": 0, "relu2": 1}
+MOE_PAIRS_PER_LAUNCH = 8192
 
 
 def moe_experts(h, gate_up, down, ids, weights, y, out, gate_max, up_min, up_max, alpha, up_shift, weight_on_input=True,
@@ -1030,6 +1035,13 @@ def moe_experts(h, gate_up, down, ids, weights, y, out, gate_max, up_min, up_max
     _need(per_pair, "per_pair", torch.float32, 2)
     if tuple(per_pair.shape) != (N * top, W):
         raise KernelError(f"per_pair must be [{N * top}, {W}]")
+    most = max(1, MOE_PAIRS_PER_LAUNCH // top)                  # a block keeps a list of an expert's pairs in shared memory
+    if N > most:
+        for n0 in range(0, N, most):
+            r, p = slice(n0, n0 + most), slice(n0 * top, (n0 + most) * top)
+            moe_experts(h[r], gate_up, down, ids[r], weights[r], y[p], out[r], gate_max, up_min, up_max, alpha, up_shift,
+                        weight_on_input, accumulate, per_pair[p], form)
+        return
     _check(lib.tnx_moe_experts(_p(h), c_int(ld), _p(gate_up), _p(down), _p(ids), _p(weights), _p(y), _p(per_pair), _p(out),
                                c_int(N), c_int(W), c_int(F), c_int(top), c_int(E), c_float(gate_max), c_float(up_min),
                                c_float(up_max),
@@ -1131,7 +1143,7 @@ def moe_grouped(ctx, h, gate_up, down, ids, weights, out, gate_max, up_min, up_m
     moe_activation(lib, gu, y, group_of_tile, tile, gate_max, up_min, up_max, alpha, up_shift, form)
     per_pair = ctx.scratch(rows, W, torch.float32)
     gemm_tc_grouped(y, down, per_pair, group_of_tile, tile, used)
-    moe_combine(lib, per_pair, row_of_pair, weights, out, accumulate, weight_on_input)
+    moe_combine(lib, per_pair, h, row_of_pair, weights, out, accumulate, weight_on_input)
 
 
 def moe_sort_rows(lib, h, ids, weights, n_experts, tiles, tile, group_of_tile, row_of_pair, x, weight_on_input):
@@ -1149,9 +1161,9 @@ def moe_activation(lib, gu, y, group_of_tile, tile, gate_max, up_min, up_max, al
                            _stream()), "moe_act")
 
 
-def moe_combine(lib, per_pair, row_of_pair, weights, out, accumulate, weight_on_input):
+def moe_combine(lib, per_pair, h, row_of_pair, weights, out, accumulate, weight_on_input):
     N, W = out.shape
-    _check(lib.tnx_moe_combine(_p(per_pair), _p(row_of_pair), _p(weights), _p(out), c_int(N), c_int(W), c_int(weights.shape[1]),
+    _check(lib.tnx_moe_combine(_p(per_pair), _p(h), c_int(h.stride(0)), _p(row_of_pair), _p(weights), _p(out), c_int(N), c_int(W), c_int(weights.shape[1]),
                                c_int(1 if accumulate else 0), c_int(1 if weight_on_input else 0), _stream()), "moe_combine")
 
 
@@ -1594,8 +1606,8 @@ def mingru_scan(proj, z_off, x_off, g_off, state, q_start, q_len, state_slots, o
                                c_int(_is_h16(proj)), _stream()), "mingru_scan")
 
 
-def gated_activation(gate_up, out, activation):
-    """out = act(gate_up[:, :F]) * gate_up[:, F:], F = out's width."""
+def gated_activation(gate_up, out, activation, row_scale=None):
+    """out = act(gate_up[:, :F]) * gate_up[:, F:], F = out's width; row n times row_scale[n] (32-bit) where it is given."""
     lib = _lib("gated_act", gate_up, out)
     _need(gate_up, "gate_up", _FLOATS, None, contiguous=False)
     N, wide, ld = _rows_2d(gate_up, "gate_up")
@@ -1603,8 +1615,10 @@ def gated_activation(gate_up, out, activation):
     No, F, out_ld = _rows_2d(out, "out")
     if No != N or wide != 2 * F:
         raise KernelError(f"gate_up must be [{No}, {2 * F}]")
+    _f32_vec(row_scale, "row_scale", N)
     _check(lib.tnx_gated_activation(_p(gate_up), c_int(ld), _p(out), c_int(out_ld), c_int(N), c_int(F),
-                                    c_int(activation_code(activation)), c_int(_is_h16(out)), _stream()), "gated_activation")
+                                    c_int(activation_code(activation)), c_int(_is_h16(out)), _p(row_scale), _stream()),
+           "gated_activation")
 
 
 # ---------------------------------------------------------------------------------------------

@@ -1,7 +1,7 @@
 """The entry-point class of a model folder, chosen by its config.json.
 
 The reference maps `model_type` to one of its sampling classes
-(src/transformers_neuronx/modeling_auto.py:5-47).  Here the table holds OPT, Vononex, Pifelix, Tutelix, Vozirax and Resatar; another architecture
+(src/transformers_neuronx/modeling_auto.py:5-47).  Here the table holds OPT, Vononex, Pifelix, Tutelix, Vozirax, Resatar and Taborax; another architecture
 registers its own entry-point class beside its registration in config/registry.py.
 """
 from __future__ import annotations
@@ -26,6 +26,7 @@ def _ensure_builtin() -> None:
     from .tutelix import model as _tutelix  # noqa: F401  registers TutelixForSampling
     from .vozirax import model as _vozirax  # noqa: F401  registers VoziraxForSampling
     from .resatar import model as _resatar  # noqa: F401  registers ResatarForSampling
+    from .taborax import model as _taborax  # noqa: F401  registers TaboraxForSampling
 
 
 class NeuronAutoModelForCausalLM:

@@ -5,3 +5,4 @@ from . import pifelix  # noqa: F401  registers Pifelix
 from . import tutelix  # noqa: F401  registers Tutelix
 from . import vozirax  # noqa: F401  registers Vozirax
 from . import resatar  # noqa: F401  registers Resatar
+from . import taborax  # noqa: F401  registers Taborax

@@ -9,7 +9,7 @@ import torch
 
 from ..kernels import build as kbuild
 from ..kernels import ops
-from ..parts import Embedding, Head, build_block, build_part
+from ..parts import Embedding, Head, StreamJoin, build_block, build_part
 from ..parts.spec import ModelSpec
 from ..weights.loader import TensorSpec
 
@@ -23,10 +23,14 @@ class DecoderModel:
             self.blocks.append(build_block(ls.block, build_part("norm", ls.norm1), build_part("mixer", ls.mixer),
                                            build_part("norm", ls.norm2),
                                            build_part("feed_forward", ls.feed_forward), layer_spec=ls))
+        self.joins = {j: StreamJoin(j) for j in dict.fromkeys(e.join for e in spec.schedule) if j is not None}
         self.head = Head(spec.head)
         for e in spec.schedule:
             if not (0 <= e.layer < len(self.blocks)):
                 raise ValueError(f"schedule names layer {e.layer}, the model has {len(self.blocks)}")
+        for j in self.joins:
+            if j.weight.out_features != spec.hidden_size:
+                raise ValueError(f"a join of width {j.weight.out_features} in a model of width {spec.hidden_size}")
         self.device = None
         self.act_dtype = None
         self._taps: Optional[Dict[str, torch.Tensor]] = None
@@ -51,6 +55,7 @@ class DecoderModel:
         out = [self.embedding]
         for b in self.blocks:
             out += b.parts()
+        out += list(self.joins.values())
         out.append(self.head)
         return out
 
@@ -100,6 +105,8 @@ class DecoderModel:
         for b in self.blocks:
             for p in b.parts():
                 p.load(tensors, device, act_dtype)
+        for j in self.joins.values():
+            j.load(tensors, device, act_dtype)
         self.head.load(tensors, device, act_dtype, shared={self.spec.embedding.table: self.embedding.table})
 
     def parameter_bytes(self) -> int:
@@ -117,26 +124,37 @@ class DecoderModel:
         ([0, vocab] when none is wanted)."""
         N, H = ctx.n_tokens, self.spec.hidden_size
         x = ctx.empty(N, H, torch.float32)
-        first = self.blocks[self.spec.schedule[0].layer] if self.spec.schedule else None
-        want_act = any(self.blocks[e.layer].needs_act_input for e in self.spec.schedule)
-        x_act = ctx.empty(N, H) if want_act else None
-        self.embedding.forward(ctx, x, x_act if (first is not None and first.needs_act_input) else None)
-        act_current = first is not None and first.needs_act_input
+        schedule, joins = self.spec.schedule, self.joins
+        first = self.blocks[schedule[0].layer] if schedule else None
+        want_act = any(self.blocks[e.layer].needs_act_input for e in schedule)
+        x_act = ctx.empty(N, H) if (want_act or joins) else None
+        act_current = first is not None and (first.needs_act_input or bool(joins))       # x_act holds x
+        self.embedding.forward(ctx, x, x_act if act_current else None)
+        from_start = {j: part.begin(ctx, x_act) for j, part in joins.items()}
         taps = self._taps
         ctx.handed_on = None
         if taps is not None:
             taps.clear()
             taps["embedding"] = x.clone()
-        for i, e in enumerate(self.spec.schedule):
+        for i, e in enumerate(schedule):
             block = self.blocks[e.layer]
+            if e.join is not None:
+                if not act_current:
+                    ops.pick_rows(x, None, out_act=x_act)
+                joins[e.join].forward(ctx, x, x_act, from_start[e.join])
+                act_current = False
             if block.needs_act_input and not act_current:
                 ops.pick_rows(x, None, out_act=x_act)
             ctx.cache_id = e.cache
             ctx.entry_index = i
-            ctx.next_block = self.blocks[self.spec.schedule[i + 1].layer] if i + 1 < len(self.spec.schedule) else None
+            after = schedule[i + 1] if i + 1 < len(schedule) else None
+            # nothing can be prepared for a block whose input a join still changes; the join wants the stream's copy
+            ctx.next_block = self.blocks[after.layer] if after is not None and after.join is None else None
+            ctx.stream_copy = x_act if after is not None and after.join is not None and not block.needs_act_input else None
+            wanted = ctx.stream_copy is not None
             ctx.begin_entry()
             block.forward(ctx, x, x_act)
-            act_current = block.keeps_act_current
+            act_current = block.keeps_act_current or (wanted and ctx.stream_copy is None)
             if taps is not None:
                 taps[f"entry{i}"] = x.clone()
         if ctx.logit_rows is None or ctx.logit_rows.shape[0] == 0:

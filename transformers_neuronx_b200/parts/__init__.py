@@ -9,4 +9,4 @@ from . import moe   # noqa: F401  the feed-forward of routed experts
 from . import latent_attention, delta_rule   # noqa: F401  attention through latents; the gated delta rule
 from . import ssd, diff_attention   # noqa: F401  the selective state-space mixer; differential attention
 from . import selective_scan   # noqa: F401  the selective scan
-from .embedding import Embedding, Head
+from .embedding import Embedding, Head, StreamJoin

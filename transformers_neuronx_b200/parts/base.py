@@ -63,6 +63,7 @@ class StepContext:
         self.entry_index = -1                 # which schedule entry runs (set by the model)
         self.next_block = None                # the block of the entry after it, or None
         self.values_of = {}                   # cache number -> this step's projected values of that entry (mixers that share them)
+        self.stream_copy = None               # where the block that runs may leave the stream's copy in the activation type
         self.handed_on = None                 # (entry index, block, tensors...): inputs a block prepared for the next one
 
     def empty(self, rows, cols, dtype=None) -> torch.Tensor:

@@ -18,7 +18,8 @@ sandwich_norm:                                            x = x + norm1_post(mix
     a norm before and after each sublayer (the layer's spec names the two further norms).  The sublayer's result
     goes into a 32-bit buffer; one kernel normalises it, adds it to the stream and, where the next sublayer of the
     same layer follows, applies that sublayer's input norm to the new row (Norm.forward_add(..., then=norm2)).  Where
-    a layer of the same kind follows, the kernel that closes this one forms that layer's first input the same way.
+    a layer of the same kind follows, the kernel that closes this one forms that layer's first input the same way; where
+    the stream itself is wanted in the activation type next (ctx.stream_copy), it leaves the row's copy there.
 
 parallel_residual:                                        x = x + s1 * mixer(norm1(x)) + s2 * ff(norm2(x))
     both sublayers read the same x, each behind a norm of its own (one kernel forms both norms: the mean square of a row
@@ -186,7 +187,11 @@ class SandwichNormBlock(ScaledPostNormBlock):
         if isinstance(nxt, SandwichNormBlock) and type(nxt.norm1) is type(norm):
             h = ctx.carry(("sandwich", (ctx.entry_index + 1) & 1), x.shape[0], x.shape[1])
             ctx.handed_on = (ctx.entry_index + 1, nxt, h)
-        norm.forward_add(ctx, x, 1.0, out, out_f32=x, out_act=h, then=nxt.norm1 if h is not None else None)
+        copy = None
+        if h is None and ctx.stream_copy is not None:
+            copy, ctx.stream_copy = ctx.stream_copy, None          # taken: whoever asked finds the copy made
+        norm.forward_add(ctx, x, 1.0, out, out_f32=x, out_act=h if h is not None else copy,
+                         then=nxt.norm1 if h is not None else None)
 
 
 class ChannelScale(Part):

@@ -15,7 +15,7 @@ from ..weights.loader import TensorSpec
 from .base import Part, to_device, weight_to_device
 from .linear import Linear, linear_forward
 from .registry import build_part
-from .spec import EmbeddingSpec, HeadSpec
+from .spec import EmbeddingSpec, HeadSpec, StreamJoinSpec
 
 
 class Embedding(Part):
@@ -76,6 +76,45 @@ class Embedding(Part):
             self.position.embed(ctx, x)
             if x_act is not None:
                 ops.pick_rows(x, None, out_act=x_act)
+
+
+class StreamJoin(Part):
+    """x <- W [x; x0], x0 being the stream as the embedding left it, where the schedule asks for it.  W is kept as its two
+    halves: x0's product does not change from one place to the next, so it is formed once a step (32-bit) and every join is
+    one product of x with the other half, to which the epilogue adds it."""
+    graph_safe = True
+
+    def __init__(self, spec: StreamJoinSpec):
+        s = self.spec = spec
+        if s.weight.in_features != 2 * s.weight.out_features or s.weight.bias:
+            raise ValueError("a join's matrix is [hidden, 2 hidden] and has no bias")
+        self.stream = self.start = None
+
+    @property
+    def libraries(self):
+        return ("gemm_simt", "gemm_tc", "gemv", "layernorm")        # the last: a copy of the stream in the activation type
+
+    def tensor_specs(self):
+        w = self.spec.weight
+        return [TensorSpec(w.weight, (w.out_features, w.in_features), "matrix")]
+
+    def load(self, tensors, device, act_dtype):
+        name, H = self.spec.weight.weight, self.spec.weight.out_features
+        w = weight_to_device(tensors[name], device, act_dtype, name)
+        self.stream, self.start = w[:, :H].contiguous(), w[:, H:].contiguous()
+
+    def parameter_bytes(self):
+        return sum(w.numel() * w.element_size() for w in (self.stream, self.start))
+
+    def begin(self, ctx, x0_act):
+        """The part of every join that x0 alone decides."""
+        out = ctx.carry(("join", self.spec), x0_act.shape[0], x0_act.shape[1], torch.float32)
+        linear_forward(x0_act, self.start, None, out)
+        return out
+
+    def forward(self, ctx, x, x_act, from_start):
+        """x <- W_x x_act + from_start (what begin() returned); x_act is x in the activation type, in memory of its own."""
+        linear_forward(x_act, self.stream, None, x, residual=from_start)
 
 
 class Head(Part):

@@ -66,12 +66,13 @@ class GatedDenseFeedForward(FeedForward):
     def parameter_bytes(self):
         return self.gate_up.parameter_bytes() + self.down.parameter_bytes()
 
-    def forward(self, ctx, h, out, accumulate=True):
+    def forward(self, ctx, h, out, accumulate=True, row_scale=None):
+        """row_scale (32-bit [tokens]): a number per token that multiplies the result."""
         N, F = h.shape[0], self.spec.up.out_features
         gu = ctx.scratch(N, 2 * F)
         self.gate_up.forward(h, gu)
         a = ctx.scratch(N, F)
-        ops.gated_activation(gu, a, self.spec.activation)
+        ops.gated_activation(gu, a, self.spec.activation, row_scale)
         self.down.forward(a, out, residual=out if accumulate else None)
 
 

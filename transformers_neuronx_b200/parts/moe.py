@@ -1,16 +1,18 @@
 """A feed-forward of routed experts: each token runs `top` of `n_experts` small feed-forwards (gated, or
 down(relu(up x)^2) without a gate; the router may have a bias, add a correction to the scores for the choice only, restrict the choice
-to the best groups of experts, and scale the weights: parts/spec.py: RoutedFeedForwardSpec).
+to the best groups of experts, scale the weights, and choose identity experts, which return their input:
+parts/spec.py: RoutedFeedForwardSpec).
 
   z = W_router h (32-bit sums), s = sigmoid(z) or softmax(z); the `top` largest scores choose the experts
   w_j = s[e_j], or s[e_j] / sum_j s[e_j] with `renormalize`
   expert(x) = W_down (g * sigmoid(act_alpha g) * (u + up_shift)),  g = min(W_gate x, gate_limit),
               u = clamp(W_up x, -up_limit, up_limit)
   result = sum_j expert_{e_j}(w_j h)  (weight_on_input)   or   sum_j w_j expert_{e_j}(h)
-           (+ shared(h), a gated feed-forward that every token runs)
+           (+ gate * shared(h), a gated feed-forward that every token runs; gate = sigmoid(W_sg h), or 1)
 
-A shared feed-forward of the experts' own form and inner width is one more expert that every token takes with weight 1: it
-rides in the experts' products.  Any other runs as the gated feed-forward it is, behind them.
+A shared feed-forward of the experts' own form whose inner width is theirs, or a small multiple, is one or a few more
+experts that every token takes with weight `gate`: it rides in the experts' products.  Any other runs as the gated
+feed-forward it is, behind them.  The gate is one more row of the router's product either way.
 
 The experts' matrices are kept stacked, [E, 2 ff, hidden] (gate rows, then up rows) and [E, hidden, ff], in the type
 they are stored in.  A step routes on the device (no read on the host: the part is graph-safe) and then takes one of
@@ -28,7 +30,7 @@ from ..kernels import ops
 from ..weights.loader import TensorSpec
 from .base import FeedForward, to_device, weight_to_device
 from .registry import build_part, register_feed_forward
-from .spec import ExpertSpec, RoutedFeedForwardSpec
+from .spec import GatedFeedForwardSpec, RoutedFeedForwardSpec
 
 
 class RoutedExperts(FeedForward):
@@ -43,12 +45,14 @@ class RoutedExperts(FeedForward):
     # width 2816, 2 a token): a decode step of 1 / 8 / 32 requests takes 0.48 / 0.75 / 1.03 ms with it and 0.52 / 1.10 /
     # 2.54 ms with the kernels that stream the matrices through the multiply-add units, so it always runs.
     GROUPED_FROM = 1
+    FOLD_MOST = 4          # a shared feed-forward of up to so many experts' widths rides in their products
 
     def __init__(self, spec: RoutedFeedForwardSpec):
         s = self.spec = spec
-        if not (1 <= s.top <= s.n_experts) or len(s.experts) != s.n_experts:
-            raise ValueError(f"{s.top} of {s.n_experts} experts ({len(s.experts)} listed) is not a choice")
-        if s.top > 16 or s.n_experts > 1024:
+        self.n_outputs = s.n_experts + s.n_identity          # of the router
+        if s.n_experts < 1 or s.n_identity < 0 or not (1 <= s.top <= self.n_outputs) or len(s.experts) != s.n_experts:
+            raise ValueError(f"{s.top} of {s.n_experts} experts ({len(s.experts)} listed) and {s.n_identity} identity experts is not a choice")
+        if s.top > 16 or self.n_outputs > 1024:
             raise ValueError("the routing kernel takes up to 16 chosen of up to 1024 experts")
         if s.scores not in ("sigmoid", "softmax"):
             raise ValueError(f"unknown scores {s.scores!r}: sigmoid or softmax")
@@ -57,27 +61,34 @@ class RoutedExperts(FeedForward):
         self.gated = s.expert_form == "gated_swish"
         if any((e.gate is None) == self.gated for e in s.experts):
             raise ValueError(f"experts of form {s.expert_form!r} {'need' if self.gated else 'have no'} gate matrices")
-        if s.n_groups < 1 or s.n_experts % s.n_groups or not (1 <= s.keep_groups <= s.n_groups) or s.group_top < 1:
-            raise ValueError(f"{s.n_experts} experts in {s.n_groups} groups of which {s.keep_groups} are kept is not a choice")
-        if s.keep_groups * (s.n_experts // s.n_groups) < s.top:
+        if s.n_groups < 1 or self.n_outputs % s.n_groups or not (1 <= s.keep_groups <= s.n_groups) or s.group_top < 1:
+            raise ValueError(f"{self.n_outputs} experts in {s.n_groups} groups of which {s.keep_groups} are kept is not a choice")
+        if s.keep_groups * (self.n_outputs // s.n_groups) < s.top:
             raise ValueError(f"the {s.keep_groups} kept groups hold fewer than {s.top} experts")
-        if (s.correction or s.n_groups > 1) and s.scores != "sigmoid":
-            raise ValueError("a correction of the choice and groups of experts go with sigmoid scores")
+        if s.shared_gate and s.shared is None:
+            raise ValueError("a gate on the shared feed-forward needs one")
         self.shared = build_part("feed_forward", s.shared)
         sh = s.shared
-        self.folded = (sh is not None and self.gated and sh.activation == "silu" and sh.up.out_features == s.ff
+        if sh is not None and not isinstance(sh, GatedFeedForwardSpec):
+            raise ValueError("the shared feed-forward of routed experts is a gated one")
+        times = sh.up.out_features // s.ff if sh is not None and sh.up.out_features % s.ff == 0 else 0
+        self.folded = (1 <= times <= self.FOLD_MOST and self.gated and sh.activation == "silu"
                        and not (sh.gate.bias or sh.up.bias or sh.down.bias) and s.act_alpha == 1.0 and s.up_shift == 0.0
                        and s.gate_limit is None and s.up_limit is None and not s.weight_on_input
-                       and s.top < 16 and s.n_experts < 1024)
+                       and s.top + times <= 16 and self.n_outputs + times <= 1024)
+        self.always = times if self.folded else 0            # experts that every token takes
         self.router = self.gate_up = self.down = self.correction = self.router_bias = None
 
     def tensor_specs(self):
         s = self.spec
-        out = [TensorSpec(s.router, (s.n_experts, s.hidden), "matrix")]
+        E = self.n_outputs
+        out = [TensorSpec(s.router, (E, s.hidden), "matrix")]
         if s.correction:
-            out.append(TensorSpec(s.correction, (s.n_experts,), "bias"))
+            out.append(TensorSpec(s.correction, (E,), "bias"))
         if s.router_bias:
-            out.append(TensorSpec(s.router_bias, (s.n_experts,), "bias"))
+            out.append(TensorSpec(s.router_bias, (E,), "bias"))
+        if s.shared_gate:
+            out.append(TensorSpec(s.shared_gate, (1, s.hidden), "matrix"))
         for e in s.experts:
             if self.gated:
                 out.append(TensorSpec(e.gate, (s.ff, s.hidden), "matrix"))
@@ -87,6 +98,11 @@ class RoutedExperts(FeedForward):
     def load(self, tensors, device, act_dtype):
         s = self.spec
         self.router = weight_to_device(tensors[s.router], device, act_dtype, s.router)
+        if s.shared_gate:                                    # one more row of the router's product
+            gate = weight_to_device(tensors[s.shared_gate], device, act_dtype, s.shared_gate)
+            if gate.dtype != self.router.dtype:
+                self.router, gate = self.router.float(), gate.float()
+            self.router = torch.cat([self.router, gate]).contiguous()
         if s.correction:
             self.correction = to_device(tensors[s.correction], device, torch.float32)
         if s.router_bias:
@@ -95,12 +111,10 @@ class RoutedExperts(FeedForward):
             self.shared.load(tensors, device, act_dtype)
         first = weight_to_device(tensors[s.experts[0].up], device, act_dtype, s.experts[0].up)
         # gate rows, then up rows; experts without a gate: the up rows alone
-        experts = s.experts
-        if self.folded:
-            experts += (ExpertSpec(s.shared.gate.weight, s.shared.up.weight, s.shared.down.weight),)
-        self.gate_up = torch.empty((len(experts), (2 if self.gated else 1) * s.ff, s.hidden), dtype=first.dtype, device=device)
-        self.down = torch.empty((len(experts), s.hidden, s.ff), dtype=first.dtype, device=device)
-        for i, e in enumerate(experts):
+        n_mats = s.n_experts + self.always
+        self.gate_up = torch.empty((n_mats, (2 if self.gated else 1) * s.ff, s.hidden), dtype=first.dtype, device=device)
+        self.down = torch.empty((n_mats, s.hidden, s.ff), dtype=first.dtype, device=device)
+        for i, e in enumerate(s.experts):
             mats = ((e.gate, self.gate_up[i, :s.ff]), (e.up, self.gate_up[i, s.ff:]), (e.down, self.down[i])) if self.gated \
                 else ((e.up, self.gate_up[i]), (e.down, self.down[i]))
             for name, dst in mats:
@@ -108,6 +122,17 @@ class RoutedExperts(FeedForward):
                 if w.dtype != first.dtype:
                     raise ValueError(f"{name} is stored as {w.dtype}, the other experts' matrices as {first.dtype}")
                 dst.copy_(w)
+        if self.folded:                                      # slices of the shared feed-forward's inner width
+            sh = s.shared
+            whole = [weight_to_device(tensors[l.weight], device, act_dtype, l.weight) for l in (sh.gate, sh.up, sh.down)]
+            for w, l in zip(whole, (sh.gate, sh.up, sh.down)):
+                if w.dtype != first.dtype:
+                    raise ValueError(f"{l.weight} is stored as {w.dtype}, the experts' matrices as {first.dtype}")
+            for j in range(self.always):
+                i, part = s.n_experts + j, slice(j * s.ff, (j + 1) * s.ff)
+                self.gate_up[i, :s.ff].copy_(whole[0][part])
+                self.gate_up[i, s.ff:].copy_(whole[1][part])
+                self.down[i].copy_(whole[2][:, part])
 
     def parameter_bytes(self):
         return sum(t.numel() * t.element_size() for t in (self.router, self.gate_up, self.down, self.correction, self.router_bias)
@@ -117,19 +142,21 @@ class RoutedExperts(FeedForward):
         """Bytes of weights a step of n_tokens is expected to read: every expert once that some token chooses, with
         tokens that choose independently and evenly."""
         s = self.spec
-        used = s.n_experts * (1.0 - (1.0 - s.top / s.n_experts) ** n_tokens)
+        used = s.n_experts * (1.0 - (1.0 - s.top / self.n_outputs) ** n_tokens)
         per = (self.gate_up[0].numel() + self.down[0].numel()) * self.gate_up.element_size()
-        shared = 0 if self.shared is None else (per if self.folded else self.shared.parameter_bytes())
+        shared = 0 if self.shared is None else (per * self.always if self.folded else self.shared.parameter_bytes())
         return int(self.router.numel() * self.router.element_size() + used * per) + shared
 
     def forward(self, ctx, h, out, accumulate=True):
         s, N = self.spec, h.shape[0]
-        always = 1 if self.folded else 0
+        always = self.always
+        gate = ctx.scratch(1, N, torch.float32).view(-1) if s.shared_gate and not self.folded else None
         ids = ctx.scratch(N, s.top + always, torch.int32)
         weights = ctx.scratch(N, s.top + always, torch.float32)
         ops.moe_route(h, self.router, ctx.token_request, ids, weights, s.top, softmax_scores=s.scores == "softmax",
                       renormalize=s.renormalize, correction=self.correction, n_groups=s.n_groups, keep_groups=s.keep_groups,
-                      group_top=s.group_top, renorm_eps=s.renorm_eps, weight_scale=s.weight_scale, bias=self.router_bias, always=always)
+                      group_top=s.group_top, renorm_eps=s.renorm_eps, weight_scale=s.weight_scale, bias=self.router_bias, always=always,
+                      n_identity=s.n_identity, gated=bool(s.shared_gate), gate_out=gate)
         inf = math.inf
         limits = (s.gate_limit if s.gate_limit is not None else inf, -s.up_limit if s.up_limit is not None else -inf,
                   s.up_limit if s.up_limit is not None else inf)
@@ -143,7 +170,10 @@ class RoutedExperts(FeedForward):
                             weight_on_input=s.weight_on_input, accumulate=accumulate,
                             per_pair=ctx.scratch(pairs, s.hidden, torch.float32), form=s.expert_form)
         if self.shared is not None and not self.folded:
-            self.shared.forward(ctx, h, out)
+            if gate is None:
+                self.shared.forward(ctx, h, out)
+            else:
+                self.shared.forward(ctx, h, out, row_scale=gate)
 
 
 register_feed_forward("routed_experts", RoutedExperts)

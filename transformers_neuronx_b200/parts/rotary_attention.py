@@ -5,6 +5,7 @@
   q, k: rotated by position on the first rotary.dims dims of each head (dim i with dim i + dims/2)
   score(i, j) = scale * head_scale[h] * <q_i, k_j> - r1[h] ln(1 + r2[h] (i - j)) (the distance bias where the spec names
       its two tensors), causal; with a window, the last `window` positions and the first `keep_first` ones; softmax in 32-bit
+  sink: one more key of a fixed score and without a value, exp(sink) more in the softmax's denominator
   rotate_values: v_j is turned by its position j over all v_dim dims before it is cached, and each head's
       output at position i is turned back by i: the sum then holds the values turned by j - i
   value mixing: the cached values are (1 - lambda) v + lambda v', v' the same tokens' values as an earlier entry of the
@@ -22,6 +23,8 @@ tcgen05 prefill, split-KV decode with its own cache append, the 32-bit kernel in
 is folded into q in 32-bit before q is rounded.
 """
 from __future__ import annotations
+
+import math
 
 import torch
 
@@ -62,6 +65,8 @@ class RotaryAttention(FusableMixer):
             raise ValueError("a distance bias needs both of its tensors")
         if s.keep_first and not s.window:
             raise ValueError("first tokens are kept beside a window; without one every position is visible")
+        if s.sink is not None and not math.isfinite(s.sink):
+            raise ValueError(f"the sink's score must be a finite number, got {s.sink}")
         if s.gate is not None:
             want = s.n_heads * (1 if s.gate_per_head else s.v_dim)
             if s.gate.out_features != want:
@@ -156,7 +161,7 @@ class RotaryAttention(FusableMixer):
                   and inner_out.dtype == q.dtype and inner_out.stride(0) % 8 == 0 and inner_out.data_ptr() % 16 == 0)
         att = inner_out if direct else ctx.scratch(N, H * D)
         ops.attention(ctx, g, q, cache, att, H, s.scale, s.window or 0, new_kv=(k, v, ctx.slot_mapping[g]),
-                      keep_first=s.keep_first, bias=self.bias)
+                      keep_first=s.keep_first, bias=self.bias, sink=s.sink)
         if not direct:
             ops.rotary_unrotate(att, ctx.token_request, ctx.positions, self.inv_freq_v, out_scale, inner_out, H, s.v_dim, D,
                                 gate=gate)

@@ -129,6 +129,7 @@ class RotaryAttentionSpec:
     # the projected values are kept for the entries that name this one.
     value_mix: Optional[str] = None
     value_source: Optional[int] = None
+    sink: Optional[float] = None     # one more key of this score and without a value: exp(sink) more in every softmax's denominator
 
 
 @dataclass(frozen=True)
@@ -389,17 +390,21 @@ class RoutedFeedForwardSpec:
     down(g * sigmoid(act_alpha g) * (u + up_shift)) with g = min(gate(x), gate_limit) and u = clamp(up(x), +-up_limit);
     the weight multiplies the expert's input x = w h (`weight_on_input`) or its output.
     With `expert_form` 'relu2' an expert has no gate: down(relu(up(x))^2).
-    Routing options (sigmoid scores): `correction` names a tensor [n_experts] that is added to the scores for the CHOICE
+    Routing options: `correction` names a tensor [n_experts] that is added to the scores for the CHOICE
     only (the weights stay the uncorrected scores); with `n_groups` > 1 the experts form equal groups of neighbours, a
     group's score is the sum of its `group_top` largest choice scores, and only experts of the `keep_groups` best groups
     can be chosen; the weights are divided by (their sum + renorm_eps) with `renormalize`, then multiplied by
-    `weight_scale`."""
+    `weight_scale`.
+    `n_identity` further outputs of the router, behind those of the experts, are identity experts: chosen like any other
+    (groups are formed over all of them), they return their input and have no tensors.
+    `shared` is a feed-forward that every token runs, added to the chosen experts'; `shared_gate` names a tensor
+    [1, hidden] whose product's sigmoid, one number per token, multiplies it."""
     kind: str                        # 'routed_experts'
     hidden: int
     ff: int
     n_experts: int
     top: int
-    router: str = None               # tensor [n_experts, hidden]
+    router: str = None               # tensor [n_experts + n_identity, hidden]
     experts: Tuple[ExpertSpec, ...] = ()
     scores: str = "sigmoid"          # 'sigmoid' | 'softmax'
     renormalize: bool = False
@@ -416,7 +421,9 @@ class RoutedFeedForwardSpec:
     renorm_eps: float = 0.0
     weight_scale: float = 1.0
     router_bias: Optional[str] = None    # tensor [n_experts], added to the router's logits
-    shared: Optional[GatedFeedForwardSpec] = None   # a feed-forward that every token runs, added to the chosen experts'
+    shared: Optional[GatedFeedForwardSpec] = None
+    shared_gate: Optional[str] = None
+    n_identity: int = 0
 
 
 @dataclass(frozen=True)
@@ -464,9 +471,16 @@ class HeadSpec:
 
 
 @dataclass(frozen=True)
+class StreamJoinSpec:
+    """x <- W [x; x0] ahead of a schedule entry, x0 being the stream as the embedding left it."""
+    weight: LinearSpec               # [hidden, 2 hidden], x's columns first; no bias
+
+
+@dataclass(frozen=True)
 class ScheduleEntry:
     layer: int                       # index into ModelSpec.layers
     cache: int                       # which cache its mixer uses; entries may share one
+    join: Optional[StreamJoinSpec] = None    # entries with equal joins share its weights
 
 
 @dataclass(frozen=True)
