@@ -25,6 +25,9 @@ closest design here (paged attention beside a recurrence with a state of fixed s
 reads another's keys and values, gated and routed feed-forwards side by side with the mixers) beside Tutelix.
 `--workload resatar`: the Resatar decoder (attention with mixed values, windowed attention with a distance bias beside
 lightning attention, a selective scan, dense and routed feed-forwards with a shared expert) beside Vozirax.
+`--workload taborax`: the Taborax decoder (attention through latents, attention with a sink whose values are its keys, a
+squared-relu feed-forward, routed experts with identity experts and a gated shared one, a looped stack) beside Tutelix (the
+same two kinds of attention) and Resatar (routed experts with a shared one).
 """
 from __future__ import annotations
 
@@ -497,6 +500,31 @@ def resatar_config(size):
             "max_positions": CONTEXT, "layers": layers}
 
 
+# ---- the Taborax decoder beside Tutelix and Resatar at equal sizes -------------------------------------
+# Heads of 128 dims; latents of 128 numbers a position (a cache row of 128, as in the decoder beside it) behind a query latent
+# of 3/8 the width; a quarter as many key heads with half of each head rotated; a feed-forward of 4x the width, or sixteen
+# experts of half the width and four identity experts in four groups, two kept, of which a token runs four beside a shared
+# expert twice as wide behind a gate (5.2 experts' parameters a token: those of the dense layer).  "loop": the first two layers
+# run twice, each pass behind a join with the embedding output.
+TABORAX_SIZES = {"2048": dict(width=2048, heads=16, kv=4), "4096": dict(width=4096, heads=32, kv=8),
+                 "2048loop": dict(width=2048, heads=16, kv=4, loop={"start": 0, "stop": 2, "times": 2})}
+TABORAX_LAYERS = ("latent_attention + dense", "attention + moe", "latent_attention + moe", "attention + moe")
+
+
+def taborax_config(size):
+    z = TABORAX_SIZES[size]
+    W, H = z["width"], z["heads"]
+    lat = {"heads": H, "dim": 128, "vdim": 128, "q_rank": 3 * W // 8, "kv_rank": 128, "scale": 128 ** -0.5}
+    att = {"heads": H, "kv_heads": z["kv"], "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "rot": {"dims": 64, "base": 5e5}}
+    moe = {"kind": "moe", "expert": {"ff": W // 2}, "shared": {"ff": W},
+           "router": {"experts": 16, "identity": 4, "top": 4, "groups": {"count": 4, "keep": 2}}}
+    layers = [{"type": "latent_attention", "mixer": lat, "mlp": {"kind": "dense", "ff": 4 * W}}, {"type": "attention", "mixer": att, "mlp": moe},
+              {"type": "latent_attention", "mixer": lat, "mlp": moe}, {"type": "attention", "mixer": att, "mlp": moe}]
+    d = {"architecture": "Taborax", "vocab": 50272, "width": W, "norm": {"eps": 1e-5}, "init_std": 0.02, "max_positions": CONTEXT,
+         "layers": layers}
+    return dict(d, loop=z["loop"]) if "loop" in z else d
+
+
 def build_vononex(size, dtype="bfloat16", config=None):
     import torch
     from transformers_neuronx_b200.config import config_from_dict
@@ -515,12 +543,16 @@ def build_vononex(size, dtype="bfloat16", config=None):
 
 
 def step_bytes(model, batch, ctx, tables_bytes):
-    """Bytes one decode step has to move: every weight once (of the embedding table only the batch's rows), the
+    """Bytes one decode step has to move: every weight once a run (of the embedding table only the batch's rows), the
     live requests' pages, and every recurrent state read and written."""
     n = model.parameter_bytes() - tables_bytes
     for part in model.all_parts():                 # routed experts: only those that the batch's tokens are expected to choose
         if hasattr(part, "step_bytes"):
             n -= part.parameter_bytes() - part.step_bytes(batch)
+    runs = [e.layer for e in model.spec.schedule]      # a layer that runs again reads its weights again
+    for i in set(runs):
+        for part in model.blocks[i].parts():
+            n += (runs.count(i) - 1) * (part.step_bytes(batch) if hasattr(part, "step_bytes") else part.parameter_bytes())
     for need in model.cache_needs().values():
         if hasattr(need, "bytes_per_page"):
             n += batch * ctx * need.bytes_per_page(16, model.act_dtype) // 16
@@ -587,7 +619,13 @@ def workload_resatar(steps, warmup, sizes=None, only=None, batch=8):
                             layers=RESATAR_LAYERS, config=resatar_config, beside="vozirax")
 
 
-BESIDE_CONFIGS = {"vononex": None, "tutelix": tutelix_config, "vozirax": vozirax_config}       # the designs that can stand beside another (None: Vononex's own)
+def workload_taborax(steps, warmup, sizes=None, only=None, batch=8):
+    """workload_vononex for the Taborax decoder, with Tutelix and Resatar at the same width beside it."""
+    return workload_vononex(steps, warmup, sizes or ["2048", "4096", "2048loop"], only, batch, design="taborax", table=TABORAX_SIZES,
+                            layers=TABORAX_LAYERS, config=taborax_config, beside=("tutelix", "resatar"))
+
+
+BESIDE_CONFIGS = {"vononex": None, "tutelix": tutelix_config, "vozirax": vozirax_config, "resatar": resatar_config}       # the designs that can stand beside another (None: Vononex's own)
 
 
 def workload_vononex(steps, warmup, sizes=None, only=None, batch=8, design="vononex", table=None, layers=None, config=None,
@@ -611,7 +649,7 @@ def workload_vononex(steps, warmup, sizes=None, only=None, batch=8, design="vono
         z = table[size]
         opt_cfg = dict(OPT_6_7B, hidden_size=z["width"], num_attention_heads=z["heads"], ffn_dim=4 * z["width"],
                        word_embed_proj_dim=z["width"])
-        for which in (design, beside):
+        for which in (design,) + (beside if isinstance(beside, tuple) else (beside,)):
             if which == design:
                 model, cfg = build_vononex(size, config=config)
                 tables = cfg.vocab * cfg.width * 2                    # the embedding table: rows of the batch only
@@ -652,6 +690,8 @@ def extra_workload(name, steps, warmup, sizes=None, only=None, batch=8):
         res = workload_vozirax(steps, warmup, sizes, only, batch)
     elif name == "resatar":
         res = workload_resatar(steps, warmup, sizes, only, batch)
+    elif name == "taborax":
+        res = workload_taborax(steps, warmup, sizes, only, batch)
     elif name == "family":
         res = workload_family(steps, warmup, sizes)
     elif name == "sweep":
@@ -687,10 +727,10 @@ def main():
     ap.add_argument("--skip-large", action="store_true", help="leave out the OPT-13B and OPT-30B workloads")
     ap.add_argument("--dtype", default="float16", choices=["float16", "bfloat16"],
                     help="the serving type (float16 is what OPT checkpoints are stored in)")
-    ap.add_argument("--workload", default=None, choices=["decode30b", "mixed13b", "family", "sweep", "vononex", "pifelix", "tutelix", "vozirax", "resatar"],
+    ap.add_argument("--workload", default=None, choices=["decode30b", "mixed13b", "family", "sweep", "vononex", "pifelix", "tutelix", "vozirax", "resatar", "taborax"],
                     help="run one of the further workloads instead of the default line")
     ap.add_argument("--sizes", default=None, help="for --workload family: comma-separated sizes (default: all of 125m .. 66b); for --workload vononex: "
-                    "widths (2048, 4096); for --workload tutelix: 2048, 4096, 2048wide; for --workload vozirax and resatar: 2048, 4096")
+                    "widths (2048, 4096); for --workload tutelix: 2048, 4096, 2048wide; for --workload vozirax and resatar: 2048, 4096; for --workload taborax: 2048, 4096, 2048loop")
     ap.add_argument("--only", default=None, choices=["decode", "prefill"],
                     help="run just this part and print its time (for profiling a small case)")
     a = ap.parse_args()
