@@ -166,8 +166,8 @@ def test_routing(E, identity, top, groups, always, gated, W):
 
 EXPERTS = [(7, 3, 24, 2, (3, 2), 48, 72, 5, torch.float32), (7, 3, 24, 2, (3, 2), 48, 72, 200, torch.float32),
            (4, 2, 36, 4, None, 30, 72, 9, torch.float32), (5, 2, 40, 1, None, None, 72, 9, torch.float32),
-           (12, 4, 64, 4, (4, 2), 64, 256, 1, torch.bfloat16), (12, 4, 64, 4, (4, 2), 64, 256, 300, torch.bfloat16),
-           (6, 2, 32, 2, None, 128, 256, 40, torch.bfloat16), (8, 1, 96, 0, (2, 1), 160, 256, 40, torch.bfloat16),
+           (12, 4, 64, 4, (4, 2), 64, 256, 1, torch.bfloat16), (12, 4, 64, 4, (4, 2), 64, 256, 300, torch.bfloat16), (12, 4, 64, 4, (4, 2), 64, 256, 600, torch.bfloat16),
+           (6, 2, 32, 2, None, 128, 256, 40, torch.bfloat16), (6, 2, 32, 2, None, 128, 256, 515, torch.bfloat16), (8, 1, 96, 0, (2, 1), 160, 256, 40, torch.bfloat16),
            (1, 1, 20, 1, None, 20, 100, 33, torch.bfloat16), (3, 2, 12, 3, (6, 4), 36, 100, 7, torch.bfloat16),
            (2, 4, 32, 6, None, 32, 64, 50, torch.bfloat16)]
 
@@ -190,14 +190,16 @@ def test_experts_identity_experts_and_a_gated_shared_one(E, top, ff, identity, g
     plain = {k[2:]: v.double() for k, v in t.items()}
     want = BP.experts(h.double(), plain, "", mlp)
     hs = torch.cat([h, torch.zeros(1, W, dtype=dtype)]).to(DEV)
-    for most in (8192, 7 * (top + part.always)):
+    # as many tokens choose it; the few-pairs launches of the 32-bit form; the folded shared expert as dense products
+    for most, apart in ((8192, type(part).APART_FROM), (7 * (top + part.always), 1)):
         monkeypatch.setattr(ops, "MOE_PAIRS_PER_LAUNCH", most)
+        monkeypatch.setattr(type(part), "APART_FROM", apart)
         ctx = _step_context(N, dtype, pad=1)
         for accumulate in (False, True):
             out = torch.full((N + 1, W), 1.0, device=DEV)
             part.forward(ctx, hs, out, accumulate=accumulate)
             _close(out[:N], want + (1.0 if accumulate else 0.0), 1e-5 if dtype == torch.float32 else 2e-2)
-            if shared is None or part.folded:
+            if shared is None or (part.folded and (apart > N or part.shared_down is None or W % 8 or ff % 8)):
                 assert float((out[N] - 1.0).abs().max()) == 0.0           # the padded row is left alone
             ctx.begin_entry()
 

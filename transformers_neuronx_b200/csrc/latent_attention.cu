@@ -11,7 +11,8 @@
 //     c   = x / sqrt(mean(x^2) + eps) * wkv -> key row and value row
 //     r turned by p (pairs (2i, 2i + 1) when interleaved, else (i, i + dr/2); angle p * inv_freq[i]) -> key row
 // tnx_headwise_product: out[n, h, :n_out] = sum_k in[n, h, k] * W[h, k, :]  for every token n and head h, 32-bit sums
-//   (W stored [heads, K, n_out]); a block takes one head and up to 8 tokens, so a head's matrix is read once per 8 tokens.
+//   (W stored [heads, K, n_out]); a block takes 64 outputs of one head and up to 8 tokens, so a head's matrix is read once
+//   per 8 tokens; its eight warps share the K rows (two neighbouring outputs a lane) and add their sums up in a fixed order.
 //   With rot_dims > 0 it also carries the head's rotated part over: in[n, h, K .. K + rot_dims) turned by the token's
 //   position to out[n, h, n_out .. n_out + rot_dims), and zeroes the head's padding up to pad_to.  do_product = 0: only
 //   that (the product was done elsewhere).
@@ -62,41 +63,74 @@ latent_prep_kernel(const T* __restrict__ proj, int ld, int col0, const int* __re
     for (int i = rkv + threadIdx.x; i < D; i += blockDim.x) vd[i] = from_float<T>(0.f);
 }
 
-constexpr int HP_TOKENS = 8;
+constexpr int HP_TOKENS = 8, HP_WARPS = 8, HP_COLS = 64, HP_AHEAD = 8;
+
+// Two neighbouring outputs of a row of W.
+__device__ __forceinline__ float2 load2(const h16* p) { return h16x2_to_float2(*(const h16x2*)p); }
+__device__ __forceinline__ float2 load2(const float* p) { return *(const float2*)p; }
 
 template <typename T>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(HP_WARPS * 32)
 headwise_product_kernel(const T* __restrict__ in, int in_ld, int in_head, const T* __restrict__ W, T* __restrict__ out,
                         int out_ld, int out_head, const int* __restrict__ token_request, const int* __restrict__ positions,
                         const float* __restrict__ inv_freq, int rot_dims, int interleaved, int pad_to, int do_product,
                         int N, int K, int n_out) {
-    extern __shared__ float xs[];                      // [HP_TOKENS][K]
+    extern __shared__ __align__(16) float xs[];        // [K][HP_TOKENS], then (same place) the warps' sums [WARPS][TOKENS][COLS]
     pdl_launch_dependents();
     pdl_wait();
-    const int h = blockIdx.x, n0 = blockIdx.y * HP_TOKENS;
+    const int h = blockIdx.x, n0 = blockIdx.y * HP_TOKENS, c0 = blockIdx.z * HP_COLS;
     const int nt = min(HP_TOKENS, N - n0);
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     if (do_product) {
-        for (int e = threadIdx.x; e < nt * K; e += blockDim.x) {
-            const int t = e / K, kk = e % K;
-            xs[e] = token_request[n0 + t] < 0 ? 0.f : to_float(in[(size_t)(n0 + t) * in_ld + (size_t)h * in_head + kk]);
+        for (int e = threadIdx.x; e < HP_TOKENS * K; e += blockDim.x) {
+            const int t = e / K, kk = e - t * K;
+            xs[kk * HP_TOKENS + t] = t < nt && token_request[n0 + t] >= 0 ? to_float(in[(size_t)(n0 + t) * in_ld + (size_t)h * in_head + kk]) : 0.f;
         }
         __syncthreads();
         const T* Wh = W + (size_t)h * K * n_out;
-        for (int c = threadIdx.x; c < n_out; c += blockDim.x) {
-            float acc[HP_TOKENS];
+        const int c = c0 + 2 * lane;
+        const bool pair = n_out % 2 == 0;              // then both outputs exist or neither, and a load of two is aligned
+        float acc[HP_TOKENS][2];
 #pragma unroll
-            for (int t = 0; t < HP_TOKENS; ++t) acc[t] = 0.f;
-            for (int kk = 0; kk < K; ++kk) {
-                const float w = to_float(Wh[(size_t)kk * n_out + c]);
+        for (int t = 0; t < HP_TOKENS; ++t) acc[t][0] = acc[t][1] = 0.f;
+        for (int k0 = warp; k0 < K; k0 += HP_WARPS * HP_AHEAD) {
+            float2 w[HP_AHEAD];
 #pragma unroll
-                for (int t = 0; t < HP_TOKENS; ++t) acc[t] = fmaf(xs[t * K + kk], w, acc[t]);     // rows beyond nt: stale, unused
+            for (int u = 0; u < HP_AHEAD; ++u) {       // all loads before the first use
+                const int kk = k0 + u * HP_WARPS;
+                const T* src = Wh + (size_t)kk * n_out + c;
+                w[u] = make_float2(0.f, 0.f);
+                if (kk < K && c < n_out) {
+                    if (pair) w[u] = load2(src);
+                    else { w[u].x = to_float(src[0]); if (c + 1 < n_out) w[u].y = to_float(src[1]); }
+                }
             }
 #pragma unroll
-            for (int t = 0; t < HP_TOKENS; ++t)
-                if (t < nt && token_request[n0 + t] >= 0)
-                    out[(size_t)(n0 + t) * out_ld + (size_t)h * out_head + c] = from_float<T>(acc[t]);
+            for (int u = 0; u < HP_AHEAD; ++u) {
+                const int kk = k0 + u * HP_WARPS;
+                if (kk < K) {
+                    const float4 a = *(const float4*)(xs + kk * HP_TOKENS), b = *(const float4*)(xs + kk * HP_TOKENS + 4);
+                    const float xv[HP_TOKENS] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+#pragma unroll
+                    for (int t = 0; t < HP_TOKENS; ++t) { acc[t][0] = fmaf(xv[t], w[u].x, acc[t][0]); acc[t][1] = fmaf(xv[t], w[u].y, acc[t][1]); }
+                }
+            }
+        }
+        __syncthreads();                               // the inputs are done with: their place takes the sums
+#pragma unroll
+        for (int t = 0; t < HP_TOKENS; ++t)
+            *(float2*)(xs + (warp * HP_TOKENS + t) * HP_COLS + 2 * lane) = make_float2(acc[t][0], acc[t][1]);
+        __syncthreads();
+        for (int e = threadIdx.x; e < nt * HP_COLS; e += blockDim.x) {
+            const int t = e / HP_COLS, cc = e % HP_COLS;
+            if (c0 + cc >= n_out || token_request[n0 + t] < 0) continue;
+            float s = 0.f;
+#pragma unroll
+            for (int w = 0; w < HP_WARPS; ++w) s += xs[(w * HP_TOKENS + t) * HP_COLS + cc];
+            out[(size_t)(n0 + t) * out_ld + (size_t)h * out_head + c0 + cc] = from_float<T>(s);
         }
     }
+    if (blockIdx.z != 0) return;
     if (pad_to <= n_out) return;
     const int half = rot_dims / 2, pad = pad_to - n_out - rot_dims;
     for (int e = threadIdx.x; e < nt * (half + pad); e += blockDim.x) {
@@ -142,14 +176,14 @@ TNX_EXPORT int tnx_headwise_product(const void* in, int in_ld, int in_head, cons
     if (n_heads <= 0 || K <= 0 || n_out <= 0 || rot_dims < 0 || rot_dims % 2 || (rot_dims && (!inv_freq || !positions)) ||
         (pad_to > n_out && pad_to < n_out + rot_dims) || (pad_to <= n_out && rot_dims) || (do_product && !W))
         return TNX_ERR_BAD_ARG;
-    const size_t smem = do_product ? (size_t)HP_TOKENS * K * sizeof(float) : 0;
+    const size_t smem = do_product ? (size_t)HP_TOKENS * (K > HP_WARPS * HP_COLS ? K : HP_WARPS * HP_COLS) * sizeof(float) : 0;
     if (smem > 200 * 1024) return TNX_ERR_UNSUPPORTED;
-    const dim3 grid(n_heads, (n_tokens + HP_TOKENS - 1) / HP_TOKENS);
+    const dim3 grid(n_heads, (n_tokens + HP_TOKENS - 1) / HP_TOKENS, do_product ? (n_out + HP_COLS - 1) / HP_COLS : 1);
 #define HPROD(T)                                                                                                         \
     do {                                                                                                                 \
         if (smem > 48 * 1024)                                                                                            \
             cudaFuncSetAttribute(headwise_product_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);    \
-        return tnx_launch_in_order(headwise_product_kernel<T>, grid, dim3(128), smem, stream, (const T*)in, in_ld, in_head, \
+        return tnx_launch_in_order(headwise_product_kernel<T>, grid, dim3(HP_WARPS * 32), smem, stream, (const T*)in, in_ld, in_head, \
                                    (const T*)W, (T*)out, out_ld, out_head, token_request, positions, inv_freq, rot_dims, \
                                    interleaved, pad_to, do_product, n_tokens, K, n_out);                                 \
     } while (0)

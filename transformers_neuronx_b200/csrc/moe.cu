@@ -16,7 +16,7 @@
 //   token takes (or is written out, for a shared feed-forward that runs on its own)
 //
 // Kernels of this file (T: the activations' type, TW: the stored type of the experts' matrices):
-//   moe_router_kernel      a block a token: logits, scores, the top experts and their weights
+//   moe_router_kernel      a block for one token or four: logits, scores, the top experts and their weights
 //   moe_gate_up_kernel     a block per (expert, slice of the inner width): the inputs of the tokens that chose the expert
 //                          in shared memory (four at a time), a warp per inner feature, 16-byte loads along the rows
 //   moe_down_kernel        a block per (expert, slice of the width): the same for the down product, one 32-bit row per pair
@@ -52,33 +52,6 @@ template <> struct Raw8<float> {
     static constexpr int AHEAD = 2;
 };
 
-// <w, x> over K elements by one warp; every lane gets the sum.  The order of the additions depends on K alone.  A lane
-// asks for AHEAD pieces of 16 bytes before it uses the first.
-template <typename TW>
-__device__ __forceinline__ float warp_dot(const TW* __restrict__ w, const float* x, int K, int lane, bool vec) {
-    constexpr int U = Raw8<TW>::AHEAD;
-    float s = 0.f;
-    if (vec) {
-        for (int c = lane * 8; c < K; c += 256 * U) {
-            Raw8<TW> a[U];
-#pragma unroll
-            for (int u = 0; u < U; ++u) if (c + 256 * u < K) a[u].load(w + c + 256 * u);
-#pragma unroll
-            for (int u = 0; u < U; ++u) {
-                if (c + 256 * u < K) {
-                    float af[8];
-                    a[u].get(af);
-#pragma unroll
-                    for (int i = 0; i < 8; ++i) s = fmaf(af[i], x[c + 256 * u + i], s);
-                }
-            }
-        }
-    } else {
-        for (int c = lane; c < K; c += 32) s = fmaf(to_float(w[c]), x[c], s);
-    }
-    return warp_sum(s);
-}
-
 struct RouterOptions {
     const float* correction;     // [E] or null
     int n_groups, keep_groups, group_top;
@@ -91,34 +64,100 @@ struct RouterOptions {
     float* gate_out;             // [N]: where the gate goes, or null
 };
 
-template <typename T, typename TW>
-__global__ void __launch_bounds__(128)
+// <w, x_t> for TOK rows of x (shared memory, pitch `ldx`) by one warp, the weights loaded once for all of them; every lane gets
+// the sums.  The order of a row's additions depends on K alone, not on TOK.
+template <typename TW, typename T, int TOK>
+__device__ __forceinline__ void warp_dots(const TW* __restrict__ w, const T* x, int ldx, int K, int lane, bool vec, float (&s)[TOK]) {
+    constexpr int U = Raw8<TW>::AHEAD;
+#pragma unroll
+    for (int t = 0; t < TOK; ++t) s[t] = 0.f;
+    if (vec) {
+        for (int c = lane * 8; c < K; c += 256 * U) {
+            Raw8<TW> a[U];
+#pragma unroll
+            for (int u = 0; u < U; ++u) if (c + 256 * u < K) a[u].load(w + c + 256 * u);
+#pragma unroll
+            for (int u = 0; u < U; ++u) {
+                if (c + 256 * u < K) {
+                    float af[8];
+                    a[u].get(af);
+#pragma unroll
+                    for (int t = 0; t < TOK; ++t) {
+                        Raw8<T> xr;
+                        float xf[8];
+                        xr.load(x + (size_t)t * ldx + c + 256 * u);
+                        xr.get(xf);
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) s[t] = fmaf(af[i], xf[i], s[t]);
+                    }
+                }
+            }
+        }
+    } else {
+        for (int c = lane; c < K; c += 32) {
+            const float wf = to_float(w[c]);
+#pragma unroll
+            for (int t = 0; t < TOK; ++t) s[t] = fmaf(wf, to_float(x[(size_t)t * ldx + c]), s[t]);
+        }
+    }
+#pragma unroll
+    for (int t = 0; t < TOK; ++t) s[t] = warp_sum(s[t]);
+}
+
+// A block takes TOK tokens, so that the router's matrix is read once for all of them: its warps share the rows of the matrix,
+// then warp t makes the choice of token t.  One token and sixteen warps for few tokens, four tokens and eight warps for many.
+template <typename T, typename TW, int TOK, int WARPS>
+__global__ void __launch_bounds__(WARPS * 32)
 moe_router_kernel(const T* __restrict__ h, int ld, const TW* __restrict__ wr, const int* __restrict__ token_request,
-                  int* __restrict__ ids, float* __restrict__ weights, int W, int E, int top, int softmax_scores,
+                  int* __restrict__ ids, float* __restrict__ weights, int N, int W, int E, int top, int softmax_scores,
                   int renormalize, RouterOptions ro) {
-    extern __shared__ __align__(16) float sm[];            // [W] the row, [E + 1] the logits (or choice scores; the gate's), [E] the scores, [E] groups
-    float* x = sm;
-    float* z = sm + ((W + 3) & ~3);
-    float* sc = z + E + 1;
-    float* gscore = sc + E;
+    extern __shared__ __align__(16) unsigned char sm_raw[];
+    const int ldx = (W + 7) & ~7;
+    T* x = (T*)sm_raw;                                       // [TOK][ldx] the rows
+    // per token: [E + 1] the logits (or choice scores; the gate's), [E] the scores, [E] the groups' scores
+    float* per_token = (float*)(sm_raw + (size_t)TOK * ldx * sizeof(T));
     pdl_launch_dependents();
     pdl_wait();
-    const int n = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const size_t row = (size_t)n * (top + ro.always);        // where the token's experts and weights begin
-    if (token_request[n] < 0) {                              // a padded row of a captured step: no expert
-        if (threadIdx.x < top + ro.always) { ids[row + threadIdx.x] = -1; weights[row + threadIdx.x] = 0.f; }
-        if (threadIdx.x == 0 && ro.gate_out) ro.gate_out[n] = 0.f;
-        return;
+    const int n0 = blockIdx.x * TOK, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int tokens = min(TOK, N - n0);
+    const bool vec_x = W % 8 == 0 && ld % 8 == 0 && ((uintptr_t)h % 16) == 0;
+#pragma unroll
+    for (int t = 0; t < TOK; ++t) {
+        const bool there = t < tokens && token_request[n0 + t] >= 0;      // rows that are not: zeros, and no choice
+        const T* src = h + (size_t)(n0 + t) * ld;
+        if (vec_x) {
+            for (int c = threadIdx.x * 8; c < W; c += WARPS * 256) {
+                Vec8<T> v;
+                if (there) v.load(src + c); else v.zero();
+                v.store(x + (size_t)t * ldx + c);
+            }
+        } else {
+            for (int c = threadIdx.x; c < W; c += WARPS * 32) x[(size_t)t * ldx + c] = there ? src[c] : from_float<T>(0.f);
+        }
     }
-    for (int c = threadIdx.x; c < W; c += blockDim.x) x[c] = to_float(h[(size_t)n * ld + c]);
     __syncthreads();
     const bool vec = W % 8 == 0 && ((uintptr_t)wr % 16) == 0;
-    for (int e = warp; e < E + ro.gated; e += 4) {
-        const float s = warp_dot<TW>(wr + (size_t)e * W, x, W, lane, vec);
-        if (lane == 0) z[e] = s + (ro.bias && e < E ? ro.bias[e] : 0.f);
+    for (int e = warp; e < E + ro.gated; e += WARPS) {
+        float s[TOK];
+        warp_dots<TW, T, TOK>(wr + (size_t)e * W, x, ldx, W, lane, vec, s);
+        const float b = ro.bias && e < E ? ro.bias[e] : 0.f;
+        if (lane == 0) {
+#pragma unroll
+            for (int t = 0; t < TOK; ++t) per_token[(size_t)t * (3 * E + 1) + e] = s[t] + b;
+        }
     }
     __syncthreads();
-    if (warp != 0) return;
+    if (warp >= tokens) return;
+    const int n = n0 + warp;                                 // this warp's token
+    float* z = per_token + (size_t)warp * (3 * E + 1);
+    float* sc = z + E + 1;
+    float* gscore = sc + E;
+    const size_t row = (size_t)n * (top + ro.always);        // where the token's experts and weights begin
+    if (token_request[n] < 0) {                              // a padded row of a captured step: no expert
+        if (lane < top + ro.always) { ids[row + lane] = -1; weights[row + lane] = 0.f; }
+        if (lane == 0 && ro.gate_out) ro.gate_out[n] = 0.f;
+        return;
+    }
     // The choice is made on the logits: both scores grow with them, and a sigmoid that has run out of bits near 1
     // would tie experts that their logits still tell apart.  With a correction or groups the choice is made on
     // choice score = score + correction, as the designs say, and the weight is the uncorrected score.
@@ -178,9 +217,8 @@ moe_router_kernel(const T* __restrict__ h, int ld, const TW* __restrict__ wr, co
             __syncwarp();
         }
     }
-    float chosen_w[MAX_TOP];
-    int chosen[MAX_TOP];
-    float total = 0.f;
+    float my_weight = 0.f, total = 0.f;                     // lane j keeps the j-th choice
+    int my_expert = 0;
     for (int j = 0; j < top; ++j) {                         // the largest logit left; of equal ones the lowest index
         float best = -INFINITY;
         int arg = 0x7fffffff;
@@ -195,20 +233,20 @@ moe_router_kernel(const T* __restrict__ h, int ld, const TW* __restrict__ wr, co
             if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
         }
         if (arg >= E) arg = 0;                              // every score left is NaN: any expert gives NaN
-        chosen[j] = arg >= E - ro.n_identity ? IDENTITY : arg;
-        chosen_w[j] = corrected ? sc[arg] : (softmax_scores ? expf(best - mx) / sum : 1.f / (1.f + expf(-best)));
-        total += chosen_w[j];
+        const float wj = corrected ? sc[arg] : (softmax_scores ? expf(best - mx) / sum : 1.f / (1.f + expf(-best)));
+        if (lane == j) { my_expert = arg >= E - ro.n_identity ? IDENTITY : arg; my_weight = wj; }
+        total += wj;
         if (lane == 0) z[arg] = -INFINITY;
         __syncwarp();
     }
-    if (lane == 0) {
-        for (int j = 0; j < top; ++j) {
-            ids[row + j] = chosen[j];
-            weights[row + j] = (renormalize ? chosen_w[j] / (total + ro.renorm_eps) : chosen_w[j]) * ro.weight_scale;
-        }
+    if (lane < top) {
+        ids[row + lane] = my_expert;
+        weights[row + lane] = (renormalize ? my_weight / (total + ro.renorm_eps) : my_weight) * ro.weight_scale;
+    }
+    if (ro.always || ro.gate_out) {
         const float gate = ro.gated ? 1.f / (1.f + expf(-z[E])) : 1.f;
-        for (int j = 0; j < ro.always; ++j) { ids[row + top + j] = E - ro.n_identity + j; weights[row + top + j] = gate; }
-        if (ro.gate_out) ro.gate_out[n] = gate;
+        if (lane < ro.always) { ids[row + top + lane] = E - ro.n_identity + lane; weights[row + top + lane] = gate; }
+        if (lane == 0 && ro.gate_out) ro.gate_out[n] = gate;
     }
 }
 
@@ -464,19 +502,29 @@ TNX_EXPORT int tnx_moe_route(const void* h, int ld, const void* router, const in
         return TNX_ERR_BAD_ARG;
     if (n_groups > 1 && E / n_groups > 64 && group_top > 1) return TNX_ERR_UNSUPPORTED;
     const RouterOptions ro{correction, n_groups, keep_groups, group_top, renorm_eps, weight_scale, bias, always, n_identity, gated, gate_out};
-    const size_t smem = (size_t)(((W + 3) & ~3) + 3 * E + 1) * sizeof(float);
-    if (smem > 160 * 1024) return TNX_ERR_UNSUPPORTED;
+    const size_t row_bytes = (size_t)((W + 7) & ~7) * (h_h16 ? 2 : 4) + (size_t)(3 * E + 1) * sizeof(float);
+    if (row_bytes > 160 * 1024) return TNX_ERR_UNSUPPORTED;
+    const bool many = N >= 512 && 4 * row_bytes <= 100 * 1024;
+#define GO_AS(T, TW, TOK, WARPS)                                                                                        \
+    do {                                                                                                                \
+        const size_t smem = TOK * row_bytes;                                                                            \
+        if (smem > 48 * 1024)                                                                                           \
+            cudaFuncSetAttribute(moe_router_kernel<T, TW, TOK, WARPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+        return tnx_launch_in_order(moe_router_kernel<T, TW, TOK, WARPS>, dim3((N + TOK - 1) / TOK), dim3(WARPS * 32), smem, stream, \
+                                   (const T*)h, ld, (const TW*)router, token_request, ids, weights, N, W, E, top,       \
+                                   softmax_scores, renormalize, ro);                                                    \
+    } while (0)
 #define GO(T, TW)                                                                                                       \
     do {                                                                                                                \
-        if (smem > 48 * 1024) cudaFuncSetAttribute(moe_router_kernel<T, TW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
-        return tnx_launch_in_order(moe_router_kernel<T, TW>, dim3(N), dim3(128), smem, stream, (const T*)h, ld,         \
-                                   (const TW*)router, token_request, ids, weights, W, E, top, softmax_scores, renormalize, ro); \
+        if (many) GO_AS(T, TW, 4, 8);                                                                                   \
+        GO_AS(T, TW, 1, 16);                                                                                            \
     } while (0)
     if (h_h16 && w_h16) GO(h16, h16);
     if (h_h16) GO(h16, float);
     if (w_h16) GO(float, h16);
     GO(float, float);
 #undef GO
+#undef GO_AS
 }
 
 TNX_EXPORT int tnx_moe_experts(const void* h, int ld, const void* gate_up, const void* down, const int* ids,

@@ -23,30 +23,45 @@ constexpr int IDENTITY = -2;      // of a pair's expert, and then of its row: th
 __global__ void __launch_bounds__(1024)
 moe_plan_kernel(const int* __restrict__ ids, int n_pairs, int n_experts, int max_tiles, int TILE, int* __restrict__ group_of_tile,
                 int* __restrict__ row_of_pair) {
-    __shared__ int count[MAX_EXPERTS], first[MAX_EXPERTS], cursor[MAX_EXPERTS];
+    __shared__ int count[MAX_EXPERTS], first[MAX_EXPERTS], cursor[MAX_EXPERTS], used_tiles;
     pdl_launch_dependents();
     pdl_wait();
     for (int e = threadIdx.x; e < n_experts; e += blockDim.x) { count[e] = 0; cursor[e] = 0; }
     __syncthreads();
-    for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) {
-        const int e = ids[i];
-        if (e >= 0) atomicAdd(&count[e], 1);
+    const int lane = threadIdx.x & 31;
+    // the lanes of a warp that hold pairs of the same expert count them together
+    for (int i0 = 0; i0 < n_pairs; i0 += blockDim.x) {
+        const int i = i0 + threadIdx.x, e = i < n_pairs ? ids[i] : -1;
+        const unsigned same = __match_any_sync(0xffffffffu, e);
+        if (e >= 0 && lane == __ffs(same) - 1) atomicAdd(&count[e], __popc(same));
     }
     __syncthreads();
-    if (threadIdx.x == 0) {
-        int tile = 0;
-        for (int e = 0; e < n_experts; ++e) {
-            first[e] = tile * TILE;
-            const int t = (count[e] + TILE - 1) / TILE;
-            for (int j = 0; j < t && tile + j < max_tiles; ++j) group_of_tile[tile + j] = e;
-            tile += t;
+    if (threadIdx.x < 32) {                            // every expert's first tile: a running sum, 32 experts at a time
+        int before = 0;
+        for (int e0 = 0; e0 < n_experts; e0 += 32) {
+            const int e = e0 + lane, t = e < n_experts ? (count[e] + TILE - 1) / TILE : 0;
+            int upto = t;
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) { const int v = __shfl_up_sync(0xffffffffu, upto, o); if (lane >= o) upto += v; }
+            if (e < n_experts) first[e] = (before + upto - t) * TILE;
+            before += __shfl_sync(0xffffffffu, upto, 31);
         }
-        for (; tile < max_tiles; ++tile) group_of_tile[tile] = -1;
+        if (lane == 0) used_tiles = before;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < n_pairs; i += blockDim.x) {
-        const int e = ids[i];
-        row_of_pair[i] = e >= 0 ? first[e] + atomicAdd(&cursor[e], 1) : e;
+    for (int e = threadIdx.x; e < n_experts; e += blockDim.x) {
+        const int tile = first[e] / TILE, t = (count[e] + TILE - 1) / TILE;
+        for (int j = 0; j < t && tile + j < max_tiles; ++j) group_of_tile[tile + j] = e;
+    }
+    for (int tile = used_tiles + threadIdx.x; tile < max_tiles; tile += blockDim.x) group_of_tile[tile] = -1;
+    for (int i0 = 0; i0 < n_pairs; i0 += blockDim.x) {
+        const int i = i0 + threadIdx.x, e = i < n_pairs ? ids[i] : -1;
+        const unsigned same = __match_any_sync(0xffffffffu, e);
+        const int leader = __ffs(same) - 1;
+        int base = 0;
+        if (e >= 0 && lane == leader) base = first[e] + atomicAdd(&cursor[e], __popc(same));
+        base = __shfl_sync(0xffffffffu, base, leader);
+        if (i < n_pairs) row_of_pair[i] = e >= 0 ? base + __popc(same & ((1u << lane) - 1u)) : e;
     }
 }
 
@@ -85,6 +100,22 @@ moe_act_kernel(const h16* __restrict__ gu, h16* __restrict__ y, const int* __res
     if (group_of_tile[row / TILE] < 0) return;
     const h16* g = gu + (size_t)row * 2 * F;
     const h16* u = g + F;
+    if (F % 8 == 0 && !(((uintptr_t)gu | (uintptr_t)y) & 15)) {
+        for (int c = threadIdx.x * 8; c < F; c += blockDim.x * 8) {
+            Vec8<h16> gv, uv;
+            float gf[8], uf[8];
+            gv.load(g + c); uv.load(u + c);
+            gv.get(gf); uv.get(uf);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                const float g0 = fminf(gf[i], gate_max), u0 = fminf(fmaxf(uf[i], up_min), up_max);
+                gf[i] = __fdividef(g0, 1.f + __expf(-alpha * g0)) * (u0 + up_shift);      // rounded to 16 bits below
+            }
+            gv.set(gf);
+            gv.store(y + (size_t)row * F + c);
+        }
+        return;
+    }
     for (int c = threadIdx.x * 2; c < F; c += blockDim.x * 2) {
         if (c + 1 < F && F % 2 == 0) {
             const float2 gf = h16x2_to_float2(*(const h16x2*)(g + c)), uf = h16x2_to_float2(*(const h16x2*)(u + c));
@@ -125,13 +156,47 @@ moe_act_relu2_kernel(const h16* __restrict__ u, h16* __restrict__ y, const int* 
     }
 }
 
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ rows, const h16* __restrict__ h, int ld, const int* __restrict__ row_of_pair,
                    const float* __restrict__ weights, float* out, int W, int top, int accumulate, int weight_on_input) {
     pdl_launch_dependents();
     pdl_wait();
     const int n = blockIdx.x;
     if (row_of_pair[(size_t)n * top] == -1) return;               // a padded row of a captured step
+    if (W % 4 == 0 && ld % 4 == 0 && !(((uintptr_t)rows | (uintptr_t)out) & 15) && !((uintptr_t)h & 7)) {
+        // four columns a thread, the rows of four choices asked for together
+        for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * 4; c < W; c += gridDim.y * blockDim.x * 4) {
+            const float4 before = accumulate ? *(const float4*)(out + (size_t)n * W + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+            float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+            for (int j0 = 0; j0 < top; j0 += 4) {
+                float4 v[4];
+                float wt[4];
+#pragma unroll
+                for (int u = 0; u < 4; ++u) {
+                    v[u] = make_float4(0.f, 0.f, 0.f, 0.f);
+                    wt[u] = 0.f;
+                    if (j0 + u >= top) continue;
+                    const int row = row_of_pair[(size_t)n * top + j0 + u];
+                    const bool self = row == IDENTITY;
+                    wt[u] = weight_on_input && !self ? 1.f : weights[(size_t)n * top + j0 + u];
+                    if (self) {
+                        const h16x2* src = (const h16x2*)(h + (size_t)n * ld + c);
+                        const float2 a = h16x2_to_float2(src[0]), b = h16x2_to_float2(src[1]);
+                        v[u] = make_float4(a.x, a.y, b.x, b.y);
+                    } else {
+                        v[u] = *(const float4*)(rows + (size_t)row * W + c);
+                    }
+                }
+#pragma unroll
+                for (int u = 0; u < 4; ++u) {
+                    s.x = fmaf(v[u].x, wt[u], s.x); s.y = fmaf(v[u].y, wt[u], s.y);
+                    s.z = fmaf(v[u].z, wt[u], s.z); s.w = fmaf(v[u].w, wt[u], s.w);
+                }
+            }
+            *(float4*)(out + (size_t)n * W + c) = make_float4(before.x + s.x, before.y + s.y, before.z + s.z, before.w + s.w);
+        }
+        return;
+    }
     for (int c = blockIdx.y * blockDim.x + threadIdx.x; c < W; c += gridDim.y * blockDim.x) {
         float s = 0.f;
         for (int j = 0; j < top; ++j) {
@@ -181,6 +246,6 @@ TNX_EXPORT int tnx_moe_combine(const float* rows, const void* h, int ld, const i
                                int accumulate, int weight_on_input, cudaStream_t stream) {
     if (N <= 0) return 0;
     // few tokens: a slice of the width a block, so that the loads of a row are asked for together
-    return tnx_launch_in_order(moe_combine_kernel, dim3(N, N >= 256 ? 1 : (W + 511) / 512), dim3(128), 0, stream, rows, (const h16*)h, ld, row_of_pair, weights, out, W, top,
+    return tnx_launch_in_order(moe_combine_kernel, dim3(N, N >= 256 ? 1 : (W + 511) / 512), dim3(N >= 256 && W >= 1024 ? 256 : 128), 0, stream, rows, (const h16*)h, ld, row_of_pair, weights, out, W, top,
                                accumulate, weight_on_input);
 }

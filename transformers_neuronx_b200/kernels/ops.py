@@ -1607,7 +1607,8 @@ def mingru_scan(proj, z_off, x_off, g_off, state, q_start, q_len, state_slots, o
 
 
 def gated_activation(gate_up, out, activation, row_scale=None):
-    """out = act(gate_up[:, :F]) * gate_up[:, F:], F = out's width; row n times row_scale[n] (32-bit) where it is given."""
+    """out = act(gate_up[:, :F]) * gate_up[:, F:], F = out's width; times row_scale (32-bit) where it is given: a number for
+    every row, or for every so many neighbouring rows."""
     lib = _lib("gated_act", gate_up, out)
     _need(gate_up, "gate_up", _FLOATS, None, contiguous=False)
     N, wide, ld = _rows_2d(gate_up, "gate_up")
@@ -1615,9 +1616,12 @@ def gated_activation(gate_up, out, activation, row_scale=None):
     No, F, out_ld = _rows_2d(out, "out")
     if No != N or wide != 2 * F:
         raise KernelError(f"gate_up must be [{No}, {2 * F}]")
-    _f32_vec(row_scale, "row_scale", N)
+    _f32_vec(row_scale, "row_scale")
+    per = 1 if row_scale is None else N // max(1, row_scale.shape[0])
+    if row_scale is not None and row_scale.shape[0] * per != N:
+        raise KernelError(f"{N} rows cannot share {row_scale.shape[0]} factors")
     _check(lib.tnx_gated_activation(_p(gate_up), c_int(ld), _p(out), c_int(out_ld), c_int(N), c_int(F),
-                                    c_int(activation_code(activation)), c_int(_is_h16(out)), _p(row_scale), _stream()),
+                                    c_int(activation_code(activation)), c_int(_is_h16(out)), _p(row_scale), c_int(max(1, per)), _stream()),
            "gated_activation")
 
 

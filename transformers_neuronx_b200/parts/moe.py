@@ -12,7 +12,8 @@ parts/spec.py: RoutedFeedForwardSpec).
 
 A shared feed-forward of the experts' own form whose inner width is theirs, or a small multiple, is one or a few more
 experts that every token takes with weight `gate`: it rides in the experts' products.  Any other runs as the gated
-feed-forward it is, behind them.  The gate is one more row of the router's product either way.
+feed-forward it is, behind them; so does the former in a step of many tokens, where a dense product of its own is the faster
+one.  The gate is one more row of the router's product either way.
 
 The experts' matrices are kept stacked, [E, 2 ff, hidden] (gate rows, then up rows) and [E, hidden, ff], in the type
 they are stored in.  A step routes on the device (no read on the host: the part is graph-safe) and then takes one of
@@ -29,6 +30,7 @@ import torch
 from ..kernels import ops
 from ..weights.loader import TensorSpec
 from .base import FeedForward, to_device, weight_to_device
+from .linear import linear_forward
 from .registry import build_part, register_feed_forward
 from .spec import GatedFeedForwardSpec, RoutedFeedForwardSpec
 
@@ -39,12 +41,14 @@ class RoutedExperts(FeedForward):
 
     @property
     def libraries(self):
-        return ("moe", "moe_grouped", "gemm_tc") + (tuple(self.shared.libraries) if self.shared is not None and not self.folded else ())
+        apart = ("gated_act", "gemm_simt") if self.folded else ()
+        return ("moe", "moe_grouped", "gemm_tc") + apart + (tuple(self.shared.libraries) if self.shared is not None and not self.folded else ())
 
     # Rows from which the grouped tensor-core form runs in a 16-bit engine.  Measured at width 2048 (8 experts of inner
     # width 2816, 2 a token): a decode step of 1 / 8 / 32 requests takes 0.48 / 0.75 / 1.03 ms with it and 0.52 / 1.10 /
     # 2.54 ms with the kernels that stream the matrices through the multiply-add units, so it always runs.
     GROUPED_FROM = 1
+    APART_FROM = 1024      # tokens from which a folded shared feed-forward runs as dense products all the same
     FOLD_MOST = 4          # a shared feed-forward of up to so many experts' widths rides in their products
 
     def __init__(self, spec: RoutedFeedForwardSpec):
@@ -77,7 +81,7 @@ class RoutedExperts(FeedForward):
                        and s.gate_limit is None and s.up_limit is None and not s.weight_on_input
                        and s.top + times <= 16 and self.n_outputs + times <= 1024)
         self.always = times if self.folded else 0            # experts that every token takes
-        self.router = self.gate_up = self.down = self.correction = self.router_bias = None
+        self.router = self.gate_up = self.down = self.correction = self.router_bias = self.shared_down = None
 
     def tensor_specs(self):
         s = self.spec
@@ -133,6 +137,8 @@ class RoutedExperts(FeedForward):
                 self.gate_up[i, :s.ff].copy_(whole[0][part])
                 self.gate_up[i, s.ff:].copy_(whole[1][part])
                 self.down[i].copy_(whole[2][:, part])
+            if act_dtype != torch.float32:
+                self.shared_down = whole[2]                  # for steps of many tokens; the other two lie in gate_up as they are
 
     def parameter_bytes(self):
         return sum(t.numel() * t.element_size() for t in (self.router, self.gate_up, self.down, self.correction, self.router_bias)
@@ -149,8 +155,9 @@ class RoutedExperts(FeedForward):
 
     def forward(self, ctx, h, out, accumulate=True):
         s, N = self.spec, h.shape[0]
-        always = self.always
-        gate = ctx.scratch(1, N, torch.float32).view(-1) if s.shared_gate and not self.folded else None
+        apart = self.shared_down is not None and N >= self.APART_FROM and ops.moe_grouped_supported(h, self.gate_up, self.down)
+        always = 0 if apart else self.always
+        gate = ctx.scratch(1, N, torch.float32).view(-1) if s.shared_gate and always == 0 else None
         ids = ctx.scratch(N, s.top + always, torch.int32)
         weights = ctx.scratch(N, s.top + always, torch.float32)
         ops.moe_route(h, self.router, ctx.token_request, ids, weights, s.top, softmax_scores=s.scores == "softmax",
@@ -161,7 +168,8 @@ class RoutedExperts(FeedForward):
         limits = (s.gate_limit if s.gate_limit is not None else inf, -s.up_limit if s.up_limit is not None else -inf,
                   s.up_limit if s.up_limit is not None else inf)
         if N >= self.GROUPED_FROM and ops.moe_grouped_supported(h, self.gate_up, self.down):
-            ops.moe_grouped(ctx, h, self.gate_up, self.down, ids, weights, out, *limits, s.act_alpha, s.up_shift,
+            E = s.n_experts + always
+            ops.moe_grouped(ctx, h, self.gate_up[:E], self.down[:E], ids, weights, out, *limits, s.act_alpha, s.up_shift,
                             weight_on_input=s.weight_on_input, accumulate=accumulate, form=s.expert_form)
         else:
             pairs = N * (s.top + always)
@@ -169,11 +177,22 @@ class RoutedExperts(FeedForward):
             ops.moe_experts(h, self.gate_up, self.down, ids, weights, y, out, *limits, s.act_alpha, s.up_shift,
                             weight_on_input=s.weight_on_input, accumulate=accumulate,
                             per_pair=ctx.scratch(pairs, s.hidden, torch.float32), form=s.expert_form)
-        if self.shared is not None and not self.folded:
+        if apart:
+            self._shared_apart(ctx, h, out, gate)
+        elif self.shared is not None and not self.folded:
             if gate is None:
                 self.shared.forward(ctx, h, out)
             else:
                 self.shared.forward(ctx, h, out, row_scale=gate)
+
+    def _shared_apart(self, ctx, h, out, gate):
+        """The folded shared feed-forward as dense products: its slices' gate and up rows are neighbours in gate_up, so a token's
+        output is `always` rows [gate | up] of the activation kernel, whose results lie in the order of the inner width."""
+        s, N, n = self.spec, h.shape[0], self.always
+        gu, a = ctx.scratch(N, n * 2 * s.ff), ctx.scratch(N, n * s.ff)
+        linear_forward(h, self.gate_up[s.n_experts:].view(n * 2 * s.ff, s.hidden), None, gu)
+        ops.gated_activation(gu.view(N * n, 2 * s.ff), a.view(N * n, s.ff), "silu", gate)
+        linear_forward(a, self.shared_down, None, out, residual=out)
 
 
 register_feed_forward("routed_experts", RoutedExperts)
