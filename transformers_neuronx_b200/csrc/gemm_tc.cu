@@ -1587,10 +1587,13 @@ TNX_EXPORT int tnx_gemm_tc_grouped(const void* A, const void* W, void* C, int M,
     CUtensorMap mp, mq;
     if (!make_map(&mp, A, M, K, lda, TILE_P)) return TNX_ERR_UNSUPPORTED;
     // tiles of 128 x 256 where a group is wide enough: half as many activation bytes per FLOP into shared memory
-    // (measured on 8 experts of 11008 x 4096 and 4096 x 5504, 4,096 rows: 2.42 against 3.28 ms for four layers' products)
+    // (measured on 8 experts of 11008 x 4096 and 4096 x 5504, 4,096 rows: 2.42 against 3.28 ms for four layers' products).
+    // Two stages, so that two CTAs fit on an SM and one's products run while the other stores its tile: 16 experts of
+    // 2048 x 2048 and 2048 x 1024 with about 410 rows each take 100 and 77 us, against 131 and 106 with one CTA of four stages;
+    // 8 of 11008 x 4096 and 4096 x 5504 with about 1,024 rows 763 and 371 against 907 and 449.
     if (N >= 256) {
         if (!make_map(&mq, W, groups * N, K, ldw, 256)) return TNX_ERR_UNSUPPORTED;
-        return launch<256, 4, false>(mp, mq, p, dim3(M / TILE_P, (N + 255) / 256, 1), stream);
+        return launch<256, 2, false>(mp, mq, p, dim3(M / TILE_P, (N + 255) / 256, 1), stream);
     }
     if (!make_map(&mq, W, groups * N, K, ldw, 128)) return TNX_ERR_UNSUPPORTED;
     return launch<128, 6, false>(mp, mq, p, dim3(M / TILE_P, (N + 127) / 128, 1), stream);
@@ -1616,7 +1619,10 @@ TNX_EXPORT int tnx_gemm_tc_batched(const void* A, const void* W, void* C, int M,
     p.batch_w_step = N; p.batch_a_step = a_step; p.batch_c_step = c_step;
     CUtensorMap mp, mq;
     if (!make_map(&mp, A, M, batches * a_step, lda, TILE_P) || !make_map(&mq, W, batches * N, K, K, 128)) return TNX_ERR_UNSUPPORTED;
-    return launch<128, 6, false>(mp, mq, p, dim3((M + TILE_P - 1) / TILE_P, (N + 127) / 128, batches), stream);
+    // few stages, several CTAs an SM: a head's product is short, and what it takes to start it and to store it counts
+    const dim3 grid((M + TILE_P - 1) / TILE_P, (N + 127) / 128, batches);
+    if (K <= 2 * BLOCK_K) return launch<128, 2, false>(mp, mq, p, grid, stream);
+    return launch<128, 3, false>(mp, mq, p, grid, stream);
 }
 
 // The same for groups of few rows: the swapped form (the group's rows of W fill the 128-row operand, `bn` = 16, 32, 64 or
