@@ -8,7 +8,7 @@ A layer's `type` names its mixer:
   'attention'         heads, kv_heads, dim, vdim (= dim: the values are the keys), scale, rot {dims, base}
 A layer's `mlp` is {"kind": "dense", "ff": F}, or {"kind": "moe", "expert": {"ff": F}, "router": {"experts": E, "top": k,
 "groups": {"count": g, "keep": n}, "identity": i}, "shared": {"ff": S}}, or null.  The router has E + i outputs, the last i
-of which are identity experts.  `loop`: layers start .. stop - 1 run `times` times in a row with the same weights.  Every
+of which are identity experts.  `loop`: the layers from `start` up to (not with) `stop` are walked `times` times.  Every
 layer carries its own sizes, so layers of one model may differ.  Nothing has a default but `init_std` (the spread of random
 weights, used only when a folder is written from a seed) and `max_positions` (the longest request the engine admits; the
 design itself has no limit); a mechanism whose key is absent or null is not there (`loop`, `rot`, `groups`, `identity`,

@@ -9,7 +9,7 @@ times with different cache numbers, the first of each pass with a join.
   latent_attention  queries through a normalised latent; keys and values expanded per head from one normalised latent, which
                     is all the pages hold; no positions
   attention         grouped key/value heads, q and k rotated in halves over the first rot.dims dims; the values are the keys
-                    as projected; one is added to the softmax's denominator (a sink of score 0)
+                    as projected; every softmax shares its weight with an empty key of score 0 (a sink)
 
 The feed-forward is down(relu(up h)^2), or routed experts: softmax scores over experts and identity experts together, a
 correction of the choice, groups scored by their best expert, weights that are the scores as they are, and a shared expert
